@@ -395,12 +395,12 @@ def retention_scan(y, q_col, k_col, v_col, decay, k_scale, frequencies, position
 
 def _pick_weights(z, mode, scale):
     if mode == 0:
-        return torch.softmax(z, dim=0)
+        return torch.softmax(z, dim=0) * scale
     s = torch.sigmoid(z)
     return s / (s.sum() + 1e-20) * scale
 
 
-def route_experts(logits, top, act, inter, x=None, router=None, mode=0, scale=1.0):
+def route_experts(logits, top, act, inter, x=None, router=None, mode=0, scale=1.0, shared_gate=None):
     if logits is None:
         logits = x.float() @ router.float().t()
     T, n = logits.shape
@@ -412,9 +412,13 @@ def route_experts(logits, top, act, inter, x=None, router=None, mode=0, scale=1.
         chosen[t, order] = True
     scaled = act[:, :n * inter].float().view(T, n, inter) * w[:, :, None]
     act[:, :n * inter] = torch.where(chosen[:, :, None], scaled, torch.zeros_like(scaled)).reshape(T, n * inter).to(act.dtype)
+    if shared_gate is not None:
+        act[:, n * inter:] = (act[:, n * inter:].float() * torch.sigmoid(x.float() @ shared_gate)[:, None]).to(act.dtype)
 
 
-def route_topk(logits, top, ids, weights, x=None, router=None, mode=0, scale=1.0):
+def route_topk(logits, top, ids, weights, x=None, router=None, mode=0, scale=1.0, shared_gate=None, gates=None):
+    if shared_gate is not None:
+        gates.copy_(torch.sigmoid(x.float() @ shared_gate))
     if logits is None:
         logits = x.float() @ router.float().t()
     for t in range(logits.shape[0]):
@@ -441,11 +445,11 @@ def gather_picks(x, lists, counts, top, rows, where):
             r += 1
 
 
-def combine_picks(y, where, weights, shared_y, out):
+def combine_picks(y, where, weights, shared_y, out, gates=None):
     T, top = weights.shape
     acc = (weights[:, :, None] * y[where.long()].float().view(T, top, -1)).sum(dim=1)
     if shared_y is not None:
-        acc = acc + shared_y.float()
+        acc = acc + shared_y.float() * (1.0 if gates is None else gates[:, None])
     out.copy_(acc.to(out.dtype))
 
 
@@ -505,6 +509,8 @@ def head_matmul(x, x_col, x_head, m, out, out_col, out_head, mode=0, tail=0, fre
         v = a @ m[h].float()
         if mode == 2 and gate is not None:
             v = v * torch.sigmoid(gate[:, gate_col + h * outer:gate_col + (h + 1) * outer].float())
+        if mode == 3 and gate is not None:
+            v = v * torch.sigmoid(gate[:, gate_col + h:gate_col + h + 1].float())
         out[:, out_col + h * out_head:out_col + h * out_head + outer] = v.to(out.dtype)
         if mode == 1 and tail:
             r = xf[:, x_col + h * x_head + inner:x_col + h * x_head + inner + tail]
@@ -622,3 +628,63 @@ def gate_into(src, y, gate_col, mode, dst, dst_col, scale, heads, v_dim):
     elif mode == 2:
         v = v * torch.sigmoid(y[:, gate_col:gate_col + heads * v_dim].float()).view(-1, heads, v_dim)
     dst[:, dst_col:dst_col + heads * v_dim] = v.reshape(src.shape[0], -1).to(dst.dtype)
+
+
+# ---- the kernels of models whose residual is several streams side by side ----
+
+
+def embedding_pair(table, second, ids, positions, token_seq, cu_q, rows, state, weight, eps, x, mul_prev, mul_cur, status=None):
+    buckets = second.shape[0] - 1
+    x.zero_()
+    kept = state.view(-1)
+    for row, a, b in _sequences(cu_q, rows):
+        for t in range(a, b):
+            r = buckets
+            if int(positions[t]) > 0:
+                before = int(ids[t - 1]) if t > a else int(kept[row])
+                r = (before * mul_prev + int(ids[t]) * mul_cur) % buckets
+            v = table[int(ids[t])].float() + second[r].float()
+            if weight is not None:
+                v = v * torch.rsqrt((v * v).mean() + eps) * weight
+            x[t] = v
+        kept[row] = ids[b - 1]
+
+
+def streams_norm(x, delta, mix, w_out, w_in, weight, eps, out, rows=None, store=True, wide=False, dtype_of_delta=0, conv=None, tail=None,
+                 token_seq=None, seq_rows=None, status=None):
+    idx = torch.arange(x.shape[0]) if rows is None else rows.long()
+    v = x[idx]
+    if mix is not None:
+        d = (delta.sum(dim=0) if delta.dim() == 3 else delta)[idx].float()
+        v = torch.einsum("st,nsw->ntw", mix, v) + w_out[None, :, None] * d[:, None, :]
+        if store:
+            x[idx] = v
+    u = (w_in[None, :, None] * v).sum(dim=1)
+    h = u * torch.rsqrt((u * u).mean(dim=-1, keepdim=True) + eps) * weight
+    if conv is not None:
+        taps = conv.shape[0]
+        y = h + conv[-1] * h
+        for t in range(x.shape[0]):
+            if taps > 1 and int(token_seq[t]) >= 0:
+                row = int(seq_rows[int(token_seq[t])])
+                y[t] += (conv[:-1] * tail[row]).sum(dim=0)
+                tail[row] = torch.cat([tail[row], h[t:t + 1]])[1:]
+        h = y
+    out.copy_(h.to(out.dtype))
+
+
+def conv_rows(h, w, tail, cu_q, seq_rows, tiles, per_tile, out, status=None):
+    taps = w.shape[0]
+    done = {}
+    for s, first in tiles.tolist():                     # the tiles must cover every sequence's tokens, each once
+        done.setdefault(s, []).append(first)
+    for i, (row, a, b) in enumerate(_sequences(cu_q, seq_rows)):
+        assert sorted(done[i]) == list(range(0, b - a, per_tile))
+        rows = torch.cat([tail[row], h[a:b]], dim=0)
+        for t in range(b - a):
+            out[a + t] = (h[a + t] + (w * rows[t:t + taps]).sum(dim=0)).to(out.dtype)
+        tail[row] = rows[-(taps - 1):]
+
+
+def relu_square(z, out):
+    out.copy_((z.float().clamp(min=0.0) ** 2).to(out.dtype))

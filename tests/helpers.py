@@ -121,6 +121,9 @@ def plain_module(folder: str):
     if c.get("architecture") == "Geponex":
         from plain import geponex_plain
         return geponex_plain
+    if c.get("architecture") == "Laposun":
+        from plain import laposun_plain
+        return laposun_plain
     if c.get("architecture") == "Fosepel":
         from plain import fosepel_plain
         return fosepel_plain

@@ -1,6 +1,7 @@
 from .base import ConfigError, KeyReader, ModelConfig
 from .fosepel import FosepelConfig
 from .geponex import GeponexConfig
+from .laposun import LaposunConfig
 from .qwen2 import Qwen2Config
 from .sisetar import SisetarConfig
 from .vegilix import VegilixConfig

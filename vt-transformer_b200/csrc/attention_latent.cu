@@ -3,7 +3,7 @@
 // A token keeps one row of D numbers (a latent of DV numbers and a key part of D - DV numbers behind it).  Every head's
 // key is the whole row and every head's value the row's first DV numbers, so the heads of a token differ in their
 // queries only (the caller has taken them into the row's space): out[t, h] = sum_j p_j row_j[:DV],
-// p = softmax_j(scale q_{t,h} . row_j) over the keys j <= position of t.  With sinks the softmax's denominator also
+// p = softmax_j(scale q_{t,h} . row_j) over the keys j <= position of t (with a window w: the last w of them).  With sinks the softmax's denominator also
 // holds exp(sink_h): a term without a key and without a value, not scaled.
 //
 // A tile is 64 rows of (token, head): a block of keys is brought into shared memory once for all of them (two-stage
@@ -41,6 +41,7 @@ struct LatentParams {
     // leave their unnormalised sums, maxima and sums in part [n_splits, tokens, heads, DV + 2] and a second kernel merges them
     int n_splits, n_tokens;
     float* part;
+    int window;                      // 0: every key up to the token's position; w: the last w of them
 };
 
 namespace {
@@ -98,15 +99,17 @@ attention_latent_kernel(const LatentParams p) {
     const int pos_lo = p.q_start[seq] + tok0, pos_hi = pos_lo + ntok - 1;
     const int key_hi = pos_hi + 1;
     const int nblk = (key_hi + KBL - 1) / KBL;
-    int blk_lo = 0, blk_hi = nblk;
+    // the blocks begin with the one that holds the first key that the tile's first token sees
+    const int first_blk = first_visible_key(pos_lo, p.window, 0) / KBL;
+    int blk_lo = first_blk, blk_hi = nblk;
     if (p.n_splits > 1) {
-        const int per = (nblk + p.n_splits - 1) / p.n_splits;
-        blk_lo = min(nblk, (int)blockIdx.z * per);
+        const int per = (nblk - first_blk + p.n_splits - 1) / p.n_splits;
+        blk_lo = min(nblk, first_blk + (int)blockIdx.z * per);
         blk_hi = min(nblk, blk_lo + per);
     }
 
     // the two rows of this thread
-    int pos[2], tok[2], head[2];
+    int pos[2], lo[2], tok[2], head[2];
     bool valid[2];
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
@@ -115,6 +118,7 @@ attention_latent_kernel(const LatentParams p) {
         valid[i] = tk < ntok && hh < nheads;
         tok[i] = q_begin + tok0 + (valid[i] ? tk : 0);
         pos[i] = pos_lo + (valid[i] ? tk : 0);
+        lo[i] = first_visible_key(pos[i], p.window, 0);
         head[i] = head0 + (valid[i] ? hh : 0);
     }
 
@@ -159,6 +163,7 @@ attention_latent_kernel(const LatentParams p) {
         }
     }
 
+    const int open_from = first_visible_key(pos_hi, p.window, 0);      // from here on every row of the tile sees a key
     if (blk_lo < blk_hi) load_block(blk_lo, 0);
     cp_async_commit();
     for (int blk = blk_lo; blk < blk_hi; ++blk) {
@@ -222,7 +227,7 @@ attention_latent_kernel(const LatentParams p) {
         }
         // mask, running maximum and sum (log2 domain)
         float mnew[2] = {mrow[0], mrow[1]};
-        const bool open = kb + KBL - 1 <= pos_lo && rows_valid >= row_base + 16 && nheads == p.heads_per_tile;
+        const bool open = kb + KBL - 1 <= pos_lo && kb >= open_from && rows_valid >= row_base + 16 && nheads == p.heads_per_tile;
         if (open) {                                      // every row of the slab sees all of the block's keys
 #pragma unroll
             for (int j = 0; j < NJ; ++j) {
@@ -239,7 +244,7 @@ attention_latent_kernel(const LatentParams p) {
                 for (int e = 0; e < 4; ++e) {
                     const int i = e >> 1;
                     const int key = kb + j * 8 + 2 * tq + (e & 1);
-                    s[j][e] = (valid[i] && key <= pos[i]) ? s[j][e] * p.scale_log2 : -INFINITY;
+                    s[j][e] = (valid[i] && key <= pos[i] && key >= lo[i]) ? s[j][e] * p.scale_log2 : -INFINITY;
                     mnew[i] = fmaxf(mnew[i], s[j][e]);
                 }
             }
@@ -378,14 +383,14 @@ bool attention_latent_supports(int key, int v_dim) {
 cudaError_t launch_attention_latent(const void* q, int q_stride, int q_col, void* out, int out_stride, int out_col, const void* pages,
                                     const int* cu_q, const int* q_start, const int* block_table, int table_stride, const int* tiles,
                                     int n_tiles, int n_pages, int heads, int key, int v_dim, int page_size, float scale,
-                                    const float* sinks, int n_splits, float* part, int n_tokens, cudaStream_t stream) {
+                                    const float* sinks, int n_splits, float* part, int n_tokens, cudaStream_t stream, int window) {
     if (n_tiles == 0) return cudaSuccess;
     if (!attention_latent_supports(key, v_dim)) return cudaErrorInvalidValue;
     if (n_splits < 1 || n_splits > 16 || (n_splits > 1 && (tiles != nullptr || part == nullptr))) return cudaErrorInvalidValue;
     const int hpt = heads < LAT_ROWS ? heads : LAT_ROWS;
     LatentParams p = {(const __nv_bfloat16*)q, q_stride, q_col, (__nv_bfloat16*)out, out_stride, out_col, (const __nv_bfloat16*)pages,
                       cu_q, q_start, block_table, table_stride, reinterpret_cast<const int2*>(tiles), n_pages, heads, page_size, key,
-                      v_dim, scale * 1.4426950408889634f, sinks, LAT_ROWS / hpt, hpt, n_splits, n_tokens, part};
+                      v_dim, scale * 1.4426950408889634f, sinks, LAT_ROWS / hpt, hpt, n_splits, n_tokens, part, window};
     const int groups = (heads + hpt - 1) / hpt;
     if (v_dim <= 64) return launch_latent_as<64, 32, 2>(p, n_tiles, groups, stream);
     if (v_dim <= 128) return launch_latent_as<128, 32, 2>(p, n_tiles, groups, stream);

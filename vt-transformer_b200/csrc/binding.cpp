@@ -473,7 +473,8 @@ void attention_diff(const Tensor& y, int64_t q_col, Tensor& out, int64_t out_col
 
 void attention_latent(const Tensor& q, int64_t q_col, Tensor& out, int64_t out_col, const Tensor& pages, const Tensor& cu_q,
                       const Tensor& q_start, const Tensor& block_table, c10::optional<Tensor> tiles, int64_t heads, int64_t key,
-                      int64_t v_dim, double scale, c10::optional<Tensor> sinks, c10::optional<Tensor> part) {
+                      int64_t v_dim, double scale, c10::optional<Tensor> sinks, c10::optional<Tensor> part, int64_t window) {
+    TORCH_CHECK(window >= 0, "attention_latent: a window of at least one token (0: none)");
     check_cuda(q, "q"); check_cuda(out, "out"); check_cuda(pages, "pages");
     check_i32(cu_q, "cu_q"); check_i32(q_start, "q_start"); check_i32(block_table, "block_table");
     TORCH_CHECK(q.scalar_type() == torch::kBFloat16 && out.scalar_type() == torch::kBFloat16 && pages.scalar_type() == torch::kBFloat16,
@@ -518,7 +519,7 @@ void attention_latent(const Tensor& q, int64_t q_col, Tensor& out, int64_t out_c
     check_launch(vtb::launch_attention_latent(q.data_ptr(), q.size(1), q_col, out.data_ptr(), out.size(1), out_col, pages.data_ptr(),
                                               cu_q.data_ptr<int>(), q_start.data_ptr<int>(), block_table.data_ptr<int>(),
                                               block_table.size(1), tp, n_tiles, pages.size(0), heads, key, v_dim, pages.size(2),
-                                              (float)scale, sp, n_splits, pp, q.size(0), stream_of(q)), "attention_latent");
+                                              (float)scale, sp, n_splits, pp, q.size(0), stream_of(q), (int)window), "attention_latent");
 }
 
 void retention_scan(const Tensor& y, int64_t q_col, int64_t k_col, int64_t v_col, const Tensor& decay, double k_scale,
@@ -599,17 +600,28 @@ struct RouterInput {
     const float* logits = nullptr;
     const void* x = nullptr;
     const float* router = nullptr;
+    const float* shared_gate = nullptr;      // [width]: a shared expert's gate, formed from x as well
     int width = 0, tokens = 0, experts = 0, x_dtype = vtb::kF32;
 };
 
-RouterInput router_input(const c10::optional<Tensor>& logits, const c10::optional<Tensor>& x, const c10::optional<Tensor>& router, const char* who) {
+RouterInput router_input(const c10::optional<Tensor>& logits, const c10::optional<Tensor>& x, const c10::optional<Tensor>& router, const char* who,
+                         const c10::optional<Tensor>& shared_gate) {
     RouterInput r;
     if (logits.has_value()) {
         check_f32(*logits, "logits");
         TORCH_CHECK(logits->dim() == 2, who, ": logits [tokens, experts]");
         r.logits = logits->data_ptr<float>(); r.tokens = logits->size(0); r.experts = logits->size(1);
-        return r;
+        if (!shared_gate.has_value()) return r;
+        TORCH_CHECK(x.has_value() && x->dim() == 2 && x->size(0) == r.tokens && x->size(1) % 8 == 0, who, ": a shared expert's gate reads the input rows");
+        check_cuda(*x, "x");
+        r.x = x->data_ptr(); r.width = x->size(1); r.x_dtype = dtype_code(*x, "x");
     }
+    if (shared_gate.has_value()) {
+        check_f32(*shared_gate, "shared_gate");
+        TORCH_CHECK(x.has_value() && shared_gate->numel() == x->size(1), who, ": a shared expert's gate [width]");
+        r.shared_gate = shared_gate->data_ptr<float>();
+    }
+    if (r.logits != nullptr) return r;
     TORCH_CHECK(x.has_value() && router.has_value(), who, ": logits, or the input rows and the router's matrix");
     check_cuda(*x, "x"); check_f32(*router, "router");
     TORCH_CHECK(x->dim() == 2 && router->dim() == 2 && router->size(1) == x->size(1) && x->size(1) % 8 == 0, who,
@@ -620,15 +632,22 @@ RouterInput router_input(const c10::optional<Tensor>& logits, const c10::optiona
 }
 
 void route_topk(c10::optional<Tensor> logits, int64_t top, Tensor& ids, Tensor& weights, c10::optional<Tensor> x, c10::optional<Tensor> router,
-                int64_t mode, double scale) {
+                int64_t mode, double scale, c10::optional<Tensor> shared_gate, c10::optional<Tensor> gates) {
     check_i32(ids, "ids"); check_f32(weights, "weights");
-    const RouterInput r = router_input(logits, x, router, "route_topk");
+    const RouterInput r = router_input(logits, x, router, "route_topk", shared_gate);
+    float* gp = nullptr;
+    if (r.shared_gate != nullptr) {
+        TORCH_CHECK(gates.has_value(), "route_topk: a shared expert's gate goes to gates [tokens]");
+        check_f32(*gates, "gates");
+        TORCH_CHECK(gates->numel() == r.tokens, "route_topk: gates [tokens]");
+        gp = gates->data_ptr<float>();
+    }
     TORCH_CHECK(ids.dim() == 2 && ids.size(0) == r.tokens && ids.size(1) == top && weights.sizes() == ids.sizes(),
                 "route_topk: ids and weights [tokens, top]");
     TORCH_CHECK(r.experts <= 1024 && top >= 1 && top <= r.experts, "route_topk: 1 <= top <= experts <= 1024");
     c10::cuda::CUDAGuard guard(ids.device());
     check_launch(vtb::launch_route_topk(r.x_dtype, r.logits, r.x, r.router, r.width, r.tokens, r.experts, top, ids.data_ptr<int>(),
-                                        weights.data_ptr<float>(), stream_of(ids), (int)mode, (float)scale), "route_topk");
+                                        weights.data_ptr<float>(), stream_of(ids), (int)mode, (float)scale, r.shared_gate, gp), "route_topk");
 }
 
 void expert_lists(const Tensor& ids, Tensor& lists, Tensor& counts) {
@@ -651,7 +670,8 @@ void gather_picks(const Tensor& x, const Tensor& lists, const Tensor& counts, in
                                           where.data_ptr<int>(), stream_of(x)), "gather_picks");
 }
 
-void combine_picks(const Tensor& y, const Tensor& where, const Tensor& weights, c10::optional<Tensor> shared_y, Tensor& out) {
+void combine_picks(const Tensor& y, const Tensor& where, const Tensor& weights, c10::optional<Tensor> shared_y, Tensor& out,
+                   c10::optional<Tensor> gates) {
     check_cuda(y, "y"); check_cuda(out, "out"); check_i32(where, "where"); check_f32(weights, "weights");
     TORCH_CHECK(weights.dim() == 2 && out.dim() == 2 && y.dim() == 2 && out.size(0) == weights.size(0) && y.size(1) == out.size(1) &&
                 y.size(0) == where.numel() && where.numel() == weights.numel() && y.scalar_type() == out.scalar_type() && out.size(1) % 8 == 0,
@@ -662,25 +682,155 @@ void combine_picks(const Tensor& y, const Tensor& where, const Tensor& weights, 
         TORCH_CHECK(shared_y->sizes() == out.sizes() && shared_y->scalar_type() == out.scalar_type(), "combine_picks: shared_y like out");
         sp = shared_y->data_ptr();
     }
+    const float* gp = nullptr;
+    if (gates.has_value()) {
+        check_f32(*gates, "gates");
+        TORCH_CHECK(gates->numel() == out.size(0), "combine_picks: gates [tokens]");
+        gp = gates->data_ptr<float>();
+    }
     c10::cuda::CUDAGuard guard(y.device());
     check_launch(vtb::launch_combine_picks(dtype_code(y, "y"), y.data_ptr(), y.size(1), where.data_ptr<int>(), weights.data_ptr<float>(),
-                                           weights.size(1), out.size(0), sp, out.data_ptr(), stream_of(y)), "combine_picks");
+                                           weights.size(1), out.size(0), sp, out.data_ptr(), stream_of(y), gp), "combine_picks");
 }
 
 void route_experts(c10::optional<Tensor> logits, int64_t top, Tensor& act, int64_t inter, c10::optional<Tensor> x, c10::optional<Tensor> router,
-                   int64_t mode, double scale) {
+                   int64_t mode, double scale, c10::optional<Tensor> shared_gate) {
     check_cuda(act, "act");
-    const RouterInput r = router_input(logits, x, router, "route_experts");
+    const RouterInput r = router_input(logits, x, router, "route_experts", shared_gate);
     TORCH_CHECK(act.dim() == 2 && act.size(0) == r.tokens, "route_experts: act [tokens, .]");
     TORCH_CHECK(r.x == nullptr || r.x_dtype == dtype_code(act, "act"), "route_experts: x and act of one dtype");
     TORCH_CHECK(r.experts >= 1 && r.experts <= 1024 && top >= 1 && top <= r.experts, "route_experts: 1 <= top <= experts <= 1024");
     TORCH_CHECK(inter >= 0 && r.experts * inter <= act.size(1), "route_experts: experts * inter columns lie outside act");
     c10::cuda::CUDAGuard guard(act.device());
     check_launch(vtb::launch_route_experts(dtype_code(act, "act"), r.logits, r.x, r.router, r.width, r.tokens, r.experts, top, act.data_ptr(),
-                                           act.size(1), inter, stream_of(act), (int)mode, (float)scale), "route_experts");
+                                           act.size(1), inter, stream_of(act), (int)mode, (float)scale, r.shared_gate), "route_experts");
 }
 
 
+
+// ---- models whose residual is several streams side by side (streams.cu)
+
+void embedding_pair(const Tensor& table, const Tensor& second, const Tensor& ids, const Tensor& positions, const Tensor& token_seq,
+                    const Tensor& cu_q, const Tensor& rows, Tensor& state, c10::optional<Tensor> weight, double eps, Tensor& x,
+                    int64_t mul_prev, int64_t mul_cur, c10::optional<Tensor> status) {
+    check_cuda(table, "table"); check_cuda(second, "second"); check_i32(ids, "ids"); check_i32(positions, "positions");
+    check_i32(token_seq, "token_seq"); check_i32(cu_q, "cu_q"); check_i32(rows, "rows"); check_i32(state, "state"); check_f32(x, "x");
+    TORCH_CHECK(table.dim() == 2 && second.dim() == 2 && x.dim() == 3 && second.scalar_type() == table.scalar_type(),
+                "embedding_pair: two tables of one dtype, x [tokens, streams, width]");
+    const int width = table.size(1);
+    TORCH_CHECK(width % 8 == 0 && width <= 12288, "embedding_pair: width ", width, " must be a multiple of 8, at most 12288");
+    TORCH_CHECK(second.size(1) == width && x.size(2) == width && second.size(0) >= 2, "embedding_pair: tables and x of one width, a second table of at least 2 rows");
+    const int64_t n = ids.numel();
+    TORCH_CHECK(x.size(0) == n && positions.numel() == n && token_seq.numel() == n && cu_q.numel() == rows.numel() + 1 && x.size(1) >= 1,
+                "embedding_pair: a position and a sequence a token, cu_q [sequences + 1]");
+    TORCH_CHECK(mul_prev >= 0 && mul_cur >= 0 && mul_prev < (1LL << 31) && mul_cur < (1LL << 31), "embedding_pair: factors between 0 and 2^31");
+    const float* wp = nullptr;
+    if (weight.has_value()) {
+        check_f32(*weight, "weight");
+        TORCH_CHECK(weight->numel() == width, "embedding_pair: a weight [width]");
+        wp = weight->data_ptr<float>();
+    }
+    c10::cuda::CUDAGuard guard(table.device());
+    check_launch(vtb::launch_embedding_pair(dtype_code(table, "table"), table.data_ptr(), second.data_ptr(), ids.data_ptr<int>(),
+                                            positions.data_ptr<int>(), token_seq.data_ptr<int>(), cu_q.data_ptr<int>(), rows.data_ptr<int>(),
+                                            rows.numel(), state.data_ptr<int>(), state.numel(), wp, (float)eps, x.data_ptr<float>(), x.size(1),
+                                            n, width, table.size(0), second.size(0) - 1, mul_prev, mul_cur, status_ptr(status),
+                                            stream_of(table)), "embedding_pair");
+}
+
+void streams_norm(Tensor& x, c10::optional<Tensor> delta, c10::optional<Tensor> mix, c10::optional<Tensor> w_out, const Tensor& w_in,
+                  const Tensor& weight, double eps, Tensor& out, c10::optional<Tensor> rows, bool store, bool wide, int64_t dtype_of_delta,
+                  c10::optional<Tensor> conv, c10::optional<Tensor> tail, c10::optional<Tensor> token_seq, c10::optional<Tensor> seq_rows,
+                  c10::optional<Tensor> status) {
+    check_f32(x, "x"); check_f32(w_in, "w_in"); check_f32(weight, "weight"); check_cuda(out, "out");
+    TORCH_CHECK(x.dim() == 3 && out.dim() == 2, "streams_norm: x [tokens, streams, width], out [rows, width]");
+    const int n = x.size(0), S = x.size(1), width = x.size(2);
+    TORCH_CHECK(width % 8 == 0 && width <= 12288 && S >= 1 && S <= 16, "streams_norm: width a multiple of 8 up to 12288, 1 to 16 streams");
+    TORCH_CHECK(w_in.numel() == S && weight.numel() == width && out.size(1) == width, "streams_norm: w_in [streams], weight [width], out [rows, width]");
+    TORCH_CHECK(!wide || out.scalar_type() == torch::kFloat32, "streams_norm: rows in 32-bit go to a float32 out");
+    const int code = wide ? (int)dtype_of_delta : dtype_code(out, "out");
+    TORCH_CHECK(mix.has_value() == delta.has_value() && mix.has_value() == w_out.has_value(), "streams_norm: a result to add comes with mix and w_out");
+    const float *mp = nullptr, *op = nullptr, *pp = nullptr;
+    const void* dp = nullptr;
+    int n_parts = 0;
+    if (mix.has_value()) {
+        check_f32(*mix, "mix"); check_f32(*w_out, "w_out");
+        TORCH_CHECK(mix->dim() == 2 && mix->size(0) == S && mix->size(1) == S && w_out->numel() == S, "streams_norm: mix [streams, streams], w_out [streams]");
+        mp = mix->data_ptr<float>();
+        op = w_out->data_ptr<float>();
+        if (delta->dim() == 3) {
+            check_f32(*delta, "delta");
+            TORCH_CHECK(delta->size(0) >= 1 && delta->size(1) == n && delta->size(2) == width, "streams_norm: shares [shares, tokens, width]");
+            pp = delta->data_ptr<float>();
+            n_parts = delta->size(0);
+        } else {
+            check_cuda(*delta, "delta");
+            TORCH_CHECK(delta->dim() == 2 && delta->size(0) == n && delta->size(1) == width && dtype_code(*delta, "delta") == code,
+                        "streams_norm: delta [tokens, width] of the compute dtype");
+            dp = delta->data_ptr();
+        }
+    }
+    const int* rp = nullptr;
+    int n_rows = n;
+    if (rows.has_value()) {
+        check_i32(*rows, "rows");
+        rp = rows->data_ptr<int>();
+        n_rows = rows->numel();
+    }
+    TORCH_CHECK(out.size(0) == n_rows, "streams_norm: out has a row for each token asked for");
+    const float* cp = nullptr;
+    float* tp = nullptr;
+    const int *sp = nullptr, *qp = nullptr;
+    int taps = 0, state_rows = 0, n_seqs = 0;
+    if (conv.has_value()) {
+        check_f32(*conv, "conv");
+        TORCH_CHECK(conv->dim() == 2 && conv->size(1) == width && conv->size(0) >= 1 && conv->size(0) <= 16 && 2 * width * 4 <= 48 * 1024,
+                    "streams_norm: conv [1 to 16 taps, width], width up to 6144");
+        TORCH_CHECK(!rows.has_value(), "streams_norm: a convolution runs over all tokens of a step");
+        cp = conv->data_ptr<float>();
+        taps = conv->size(0);
+        if (taps > 1) {
+            TORCH_CHECK(tail.has_value() && token_seq.has_value() && seq_rows.has_value(), "streams_norm: a convolution of several taps has a tail");
+            check_f32(*tail, "tail"); check_i32(*token_seq, "token_seq"); check_i32(*seq_rows, "seq_rows");
+            TORCH_CHECK(tail->dim() == 3 && tail->size(1) == taps - 1 && tail->size(2) == width && token_seq->numel() == n,
+                        "streams_norm: tail [rows, taps - 1, width], a sequence a token");
+            tp = tail->data_ptr<float>();
+            state_rows = tail->size(0);
+            sp = token_seq->data_ptr<int>();
+            qp = seq_rows->data_ptr<int>();
+            n_seqs = seq_rows->numel();
+        }
+    }
+    c10::cuda::CUDAGuard guard(x.device());
+    check_launch(vtb::launch_streams_norm(code, x.data_ptr<float>(), n, S, width, dp, pp, n_parts, mp, op, w_in.data_ptr<float>(),
+                                          weight.data_ptr<float>(), (float)eps, wide ? nullptr : out.data_ptr(),
+                                          wide ? out.data_ptr<float>() : nullptr, rp, n_rows, store ? 1 : 0, cp, taps, tp, state_rows, sp, qp,
+                                          n_seqs, status_ptr(status), stream_of(x)), "streams_norm");
+}
+
+void conv_rows(const Tensor& h, const Tensor& w, Tensor& tail, const Tensor& cu_q, const Tensor& seq_rows, const Tensor& tiles, int64_t per_tile,
+               Tensor& out, c10::optional<Tensor> status) {
+    check_f32(h, "h"); check_f32(w, "w"); check_f32(tail, "tail"); check_i32(cu_q, "cu_q"); check_i32(seq_rows, "seq_rows");
+    check_i32(tiles, "tiles"); check_cuda(out, "out");
+    TORCH_CHECK(h.dim() == 2 && out.dim() == 2 && out.sizes() == h.sizes() && h.size(1) % 8 == 0, "conv_rows: h and out [tokens, width], width a multiple of 8");
+    TORCH_CHECK(out.data_ptr() != h.data_ptr(), "conv_rows: out must not be h");
+    const int width = h.size(1);
+    TORCH_CHECK(w.dim() == 2 && w.size(1) == width && w.size(0) >= 2 && w.size(0) <= 16, "conv_rows: w [2 to 16 taps, width]");
+    TORCH_CHECK(tail.dim() == 3 && tail.size(1) == w.size(0) - 1 && tail.size(2) == width, "conv_rows: tail [rows, taps - 1, width]");
+    TORCH_CHECK(cu_q.numel() == seq_rows.numel() + 1 && tiles.dim() == 2 && tiles.size(1) == 2 && per_tile >= w.size(0) - 1,
+                "conv_rows: cu_q [sequences + 1], tiles [n, 2] of at least taps - 1 tokens");
+    c10::cuda::CUDAGuard guard(h.device());
+    check_launch(vtb::launch_conv_rows(dtype_code(out, "out"), h.data_ptr<float>(), w.data_ptr<float>(), w.size(0), tail.data_ptr<float>(),
+                                       tail.size(0), cu_q.data_ptr<int>(), seq_rows.data_ptr<int>(), tiles.data_ptr<int>(), tiles.size(0),
+                                       per_tile, out.data_ptr(), width, status_ptr(status), stream_of(h)), "conv_rows");
+}
+
+void relu_square(const Tensor& z, Tensor& out) {
+    check_cuda(z, "z"); check_cuda(out, "out");
+    TORCH_CHECK(z.sizes() == out.sizes() && z.scalar_type() == out.scalar_type(), "relu_square: z and out of one shape and dtype");
+    c10::cuda::CUDAGuard guard(z.device());
+    check_launch(vtb::launch_relu_square(dtype_code(z, "z"), z.data_ptr(), out.data_ptr(), z.numel(), stream_of(z)), "relu_square");
+}
 
 // ---- layers with a latent for each token (latent.cu)
 
@@ -736,7 +886,7 @@ void head_matmul(const Tensor& x, int64_t x_col, int64_t x_head, const Tensor& m
     check_cuda(x, "x"); check_cuda(m, "m"); check_cuda(out, "out");
     TORCH_CHECK(x.dim() == 2 && out.dim() == 2 && m.dim() == 3 && out.size(0) == x.size(0) && out.scalar_type() == x.scalar_type(),
                 "head_matmul: x and out [tokens, .] of one dtype, m [heads, inner, outer]");
-    TORCH_CHECK(mode >= 0 && mode <= 2 && tail >= 0, "head_matmul: mode 0, 1 (a rotated tail) or 2 (a gate)");
+    TORCH_CHECK(mode >= 0 && mode <= 3 && tail >= 0, "head_matmul: mode 0, 1 (a rotated tail), 2 (a gate) or 3 (a gate a head)");
     const int heads = m.size(0), inner = m.size(1), outer = m.size(2);
     TORCH_CHECK(inner <= 1536, "head_matmul: inner sizes up to 1536");
     TORCH_CHECK(x_head >= inner + (mode == 1 ? tail : 0) && out_head >= outer + (mode == 1 ? tail : 0), "head_matmul: a head's inputs and "
@@ -759,9 +909,9 @@ void head_matmul(const Tensor& x, int64_t x_col, int64_t x_head, const Tensor& m
     int gate_stride = 0;
     if (gate.has_value()) {
         check_cuda(*gate, "gate");
-        TORCH_CHECK(mode == 2 && gate->dim() == 2 && gate->size(0) == x.size(0) && gate->scalar_type() == x.scalar_type(),
-                    "head_matmul: a gate [tokens, .] of x's dtype, with mode 2");
-        check_cols(*gate, gate_col, heads * outer, "head_matmul (gate)");
+        TORCH_CHECK(mode >= 2 && gate->dim() == 2 && gate->size(0) == x.size(0) && gate->scalar_type() == x.scalar_type(),
+                    "head_matmul: a gate [tokens, .] of x's dtype, with mode 2 or 3");
+        check_cols(*gate, gate_col, mode == 3 ? heads : heads * outer, "head_matmul (gate)");
         gp = gate->data_ptr();
         gate_stride = gate->size(1);
     }
@@ -900,7 +1050,7 @@ void gemm_tc(const Tensor& x, const Tensor& w, c10::optional<Tensor> bias, Tenso
     TORCH_CHECK(x.scalar_type() == torch::kBFloat16 && w.scalar_type() == torch::kBFloat16, "gemm_tc: x and w must be bfloat16");
     TORCH_CHECK(x.dim() == 2 && w.dim() == 2, "gemm_tc: x and w must be 2-d");
     const int m = x.size(0), k = x.size(1), n = w.size(0);
-    TORCH_CHECK(epilogue >= 0 && epilogue <= 2, "gemm_tc: epilogue must be 0 (bias), 1 (silu(gate) * up) or 2 (unadded shares)");
+    TORCH_CHECK(epilogue >= 0 && epilogue <= 3, "gemm_tc: epilogue must be 0 (bias), 1 (silu(gate) * up), 2 (unadded shares) or 3 (max(., 0)^2)");
     if (epilogue == 2) {
         TORCH_CHECK(w.size(1) == k && out.dim() == 3 && out.scalar_type() == torch::kFloat32 && out.is_contiguous() &&
                         out.size(0) == vtb::gemm_tc_shares(m, n, k) && out.size(1) == m && out.size(2) == n,
@@ -911,6 +1061,7 @@ void gemm_tc(const Tensor& x, const Tensor& w, c10::optional<Tensor> bias, Tenso
     }
     TORCH_CHECK(epilogue != 1 || (n % 16 == 0 && !bias.has_value() && out.scalar_type() == torch::kBFloat16),
                 "gemm_tc: the silu epilogue takes n % 16 == 0, no bias and a bfloat16 out");
+    TORCH_CHECK(epilogue != 3 || (!bias.has_value() && out.scalar_type() == torch::kBFloat16), "gemm_tc: epilogue 3 takes no bias and a bfloat16 out");
     TORCH_CHECK(k % 8 == 0, "gemm_tc: inner size ", k, " must be a multiple of 8 (TMA rows start on 16-byte boundaries)");
     TORCH_CHECK(((uintptr_t)x.data_ptr() & 15) == 0 && ((uintptr_t)w.data_ptr() & 15) == 0,
                 "gemm_tc: x and w must start on 16-byte boundaries");
@@ -945,7 +1096,8 @@ void gemm_tc_pair(const Tensor& x, const Tensor& w, c10::optional<Tensor> bias, 
                 "gemm_tc_pair: x, w and out must be bfloat16");
     TORCH_CHECK(x.dim() == 2 && w.dim() == 2 && out.dim() == 2, "gemm_tc_pair: x, w and out must be 2-d");
     const int m = x.size(0), k = x.size(1), n = w.size(0);
-    TORCH_CHECK(epilogue == 0 || epilogue == 1, "gemm_tc_pair: epilogue must be 0 (bias) or 1 (silu(gate) * up)");
+    TORCH_CHECK(epilogue == 0 || epilogue == 1 || epilogue == 3, "gemm_tc_pair: epilogue must be 0 (bias), 1 (silu(gate) * up) or 3 (max(., 0)^2)");
+    TORCH_CHECK(epilogue != 3 || !bias.has_value(), "gemm_tc_pair: epilogue 3 takes no bias");
     TORCH_CHECK(bn == 0 || bn == 256 || bn == 224 || bn == 192, "gemm_tc_pair: tiles of 256, 224 or 192 rows of w (0: chosen by the sizes)");
     TORCH_CHECK(w.size(1) == k && out.size(0) == m && out.size(1) == (epilogue == 1 ? n / 2 : n),
                 "gemm_tc_pair: shapes [m,k] x [n,k] -> [m,n] (or [m,n/2] with the silu epilogue)");
@@ -1238,7 +1390,19 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
     m.def("attention_diff", &attention_diff);
     m.def("attention_diff_supports", &vtb::attention_diff_supports);
     m.def("attention_diff_tile_rows", &vtb::attention_diff_tile_rows);
-    m.def("attention_latent", &attention_latent);
+    m.def("attention_latent", &attention_latent, py::arg("q"), py::arg("q_col"), py::arg("out"), py::arg("out_col"), py::arg("pages"),
+          py::arg("cu_q"), py::arg("q_start"), py::arg("block_table"), py::arg("tiles"), py::arg("heads"), py::arg("key"), py::arg("v_dim"),
+          py::arg("scale"), py::arg("sinks") = py::none(), py::arg("part") = py::none(), py::arg("window") = 0);
+    m.def("embedding_pair", &embedding_pair, py::arg("table"), py::arg("second"), py::arg("ids"), py::arg("positions"), py::arg("token_seq"),
+          py::arg("cu_q"), py::arg("rows"), py::arg("state"), py::arg("weight"), py::arg("eps"), py::arg("x"), py::arg("mul_prev"),
+          py::arg("mul_cur"), py::arg("status") = py::none());
+    m.def("streams_norm", &streams_norm, py::arg("x"), py::arg("delta"), py::arg("mix"), py::arg("w_out"), py::arg("w_in"), py::arg("weight"),
+          py::arg("eps"), py::arg("out"), py::arg("rows") = py::none(), py::arg("store") = true, py::arg("wide") = false,
+          py::arg("dtype_of_delta") = 0, py::arg("conv") = py::none(), py::arg("tail") = py::none(), py::arg("token_seq") = py::none(),
+          py::arg("seq_rows") = py::none(), py::arg("status") = py::none());
+    m.def("conv_rows", &conv_rows, py::arg("h"), py::arg("w"), py::arg("tail"), py::arg("cu_q"), py::arg("seq_rows"), py::arg("tiles"),
+          py::arg("per_tile"), py::arg("out"), py::arg("status") = py::none());
+    m.def("relu_square", &relu_square, py::arg("z"), py::arg("out"));
     m.def("attention_latent_supports", &vtb::attention_latent_supports);
     m.def("attention_latent_tile_rows", &vtb::attention_latent_tile_rows);
     m.def("retention_scan", &retention_scan, py::arg("y"), py::arg("q_col"), py::arg("k_col"), py::arg("v_col"), py::arg("decay"),
@@ -1249,9 +1413,10 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
     m.def("retention_fix", &retention_fix, py::arg("y"), py::arg("q_col"), py::arg("positions"), py::arg("frequencies"), py::arg("starts"),
           py::arg("tiles"), py::arg("decay"), py::arg("o"), py::arg("act") = 0);
     m.def("route_experts", &route_experts, py::arg("logits"), py::arg("top"), py::arg("act"), py::arg("inter"), py::arg("x") = py::none(),
-          py::arg("router") = py::none(), py::arg("mode") = 0, py::arg("scale") = 1.0);
+          py::arg("router") = py::none(), py::arg("mode") = 0, py::arg("scale") = 1.0, py::arg("shared_gate") = py::none());
     m.def("route_topk", &route_topk, py::arg("logits"), py::arg("top"), py::arg("ids"), py::arg("weights"), py::arg("x") = py::none(),
-          py::arg("router") = py::none(), py::arg("mode") = 0, py::arg("scale") = 1.0);
+          py::arg("router") = py::none(), py::arg("mode") = 0, py::arg("scale") = 1.0, py::arg("shared_gate") = py::none(),
+          py::arg("gates") = py::none());
     m.def("token_shift", &token_shift, py::arg("x"), py::arg("mu"), py::arg("state"), py::arg("cu_q"), py::arg("rows"), py::arg("token_seq"),
           py::arg("out"), py::arg("status") = py::none());
     m.def("latent_prepare", &latent_prepare, py::arg("y"), py::arg("q_col"), py::arg("q_rank"), py::arg("kv_col"), py::arg("kv_rank"),
@@ -1266,7 +1431,8 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
           py::arg("split"), py::arg("limit2"));
     m.def("expert_lists", &expert_lists);
     m.def("gather_picks", &gather_picks);
-    m.def("combine_picks", &combine_picks);
+    m.def("combine_picks", &combine_picks, py::arg("y"), py::arg("where"), py::arg("weights"), py::arg("shared_y"), py::arg("out"),
+          py::arg("gates") = py::none());
     m.def("silu_mul", &silu_mul, py::arg("gu"), py::arg("out"), py::arg("interleave") = 0);
     m.def("rope_store", &rope_store, py::arg("qkv"), py::arg("positions"), py::arg("cos_sin"), py::arg("k_cache"),
           py::arg("v_cache"), py::arg("token_seq"), py::arg("block_table"), py::arg("heads"), py::arg("kv_heads"),

@@ -41,8 +41,9 @@ SOURCES = [
     "attention_diff.cu",
     "attention_latent.cu",
     "latent.cu",
+    "streams.cu",
 ]
-HEADERS = ["common.cuh", "kernels.h", "launch.cuh", "tc_common.cuh", "gemm_epilogue.cuh", "attention_mma.cuh", "attention_decode.cuh", "attention_noalloc.h"]
+HEADERS = ["common.cuh", "kernels.h", "launch.cuh", "tc_common.cuh", "gemm_epilogue.cuh", "attention_mma.cuh", "attention_decode.cuh", "attention_noalloc.h", "look_ahead.cuh"]
 
 CUDA_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",

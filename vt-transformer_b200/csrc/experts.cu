@@ -23,7 +23,8 @@ constexpr int kRouteThreads = 128;
 
 // The `top` largest of z[0 .. experts) (the lower index among equals), by the first warp of the block: picked[k] and
 // picked_z[k] in falling order; z is used up.  Then w[e] = the pick's weight (0 for the others) if w is given: mode 0 the
-// softmax over the picked logits; mode 1 each pick's sigmoid(logit) over the picks' sum of them (+ 1e-20), times `scale`.
+// softmax over the picked logits, times `scale` (the softmax over all logits divided by the picks' sum of it is the same number);
+// mode 1 each pick's sigmoid(logit) over the picks' sum of them (+ 1e-20), times `scale`.
 __device__ __forceinline__ void pick_top(float* z, float* w, int* picked, float* picked_z, int experts, int top, int mode = 0,
                                          float scale = 1.f) {
     const int lane = threadIdx.x & 31;
@@ -64,7 +65,7 @@ __device__ __forceinline__ void pick_top(float* z, float* w, int* picked, float*
         float sum = 0.f;
         for (int k = 0; k < top; ++k) sum += expf(picked_z[k] - mx);
         for (int k = 0; k < top; ++k) {
-            const float wk = expf(picked_z[k] - mx) / sum;
+            const float wk = expf(picked_z[k] - mx) / sum * scale;
             picked_z[k] = wk;                          // from here on: the pick's weight
             if (w) w[picked[k]] = wk;
         }
@@ -74,17 +75,19 @@ __device__ __forceinline__ void pick_top(float* z, float* w, int* picked, float*
 // z[e] = logits[t, e], or, with the router's matrix [experts, width] (32-bit) and the token's input row x [width], the
 // dot product formed here in 32-bit: a warp an expert, a lane the same columns of every expert, the lanes' sums added by
 // the warp: the order depends on the width alone.
+// With a shared expert's gate (a vector [width], x given) z[experts] is its dot product with x, formed the same way.
 template <typename T>
 __device__ __forceinline__ void router_logits(float* z, const float* __restrict__ logits, const T* __restrict__ x,
-                                              const float* __restrict__ router, int width, int experts, int t) {
-    if (x == nullptr) {
+                                              const float* __restrict__ router, int width, int experts, int t,
+                                              const float* __restrict__ shared_gate) {
+    if (logits != nullptr)
         for (int e = threadIdx.x; e < experts; e += blockDim.x) z[e] = logits[(size_t)t * experts + e];
-        return;
-    }
+    if (x == nullptr) return;
+    const int from = logits != nullptr ? experts : 0, rows = experts + (shared_gate != nullptr ? 1 : 0);
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
     const T* xr = x + (size_t)t * width;
-    for (int e = warp; e < experts; e += warps) {
-        const float* rr = router + (size_t)e * width;
+    for (int e = from + warp; e < rows; e += warps) {
+        const float* rr = e < experts ? router + (size_t)e * width : shared_gate;
         float acc = 0.f;
         for (int c = lane * 8; c < width; c += 256) {
             float a[8], b[8];
@@ -101,8 +104,9 @@ __device__ __forceinline__ void router_logits(float* z, const float* __restrict_
 template <typename T>
 __global__ void __launch_bounds__(kRouteThreads)
 route_experts_kernel(const float* __restrict__ logits, const T* __restrict__ x, const float* __restrict__ router, int width,
-                     int experts, int top, T* __restrict__ act, int act_stride, int inter, int mode, float scale) {
-    __shared__ float z[kMaxExperts];          // the logits; a picked one is taken out
+                     int experts, int top, T* __restrict__ act, int act_stride, int inter, int mode, float scale,
+                     const float* __restrict__ shared_gate) {
+    __shared__ float z[kMaxExperts + 1];      // the logits (a picked one is taken out), and the shared expert's
     __shared__ float w[kMaxExperts];          // the experts' weights, zero for those not picked
     __shared__ float picked_z[kMaxExperts];
     __shared__ int picked[kMaxExperts];
@@ -110,17 +114,21 @@ route_experts_kernel(const float* __restrict__ logits, const T* __restrict__ x, 
     pdl_wait();
     const int t = blockIdx.x;
     for (int e = threadIdx.x; e < experts; e += blockDim.x) w[e] = 0.f;
-    router_logits(z, logits, x, router, width, experts, t);
+    router_logits(z, logits, x, router, width, experts, t, shared_gate);
     __syncthreads();
     pick_top(z, w, picked, picked_z, experts, top, mode, scale);
     __syncthreads();
     T* row = act + (size_t)t * act_stride;
+    if (shared_gate != nullptr) {
+        const float g = 1.f / (1.f + expf(-z[experts]));
+        for (int c = experts * inter + threadIdx.x; c < act_stride; c += blockDim.x) row[c] = from_float<T>(to_float(row[c]) * g);
+    }
     if (inter % 8 == 0 && act_stride % 8 == 0 && (reinterpret_cast<uintptr_t>(act) & 15) == 0) {
         const int per = inter / 8;
         for (int c = threadIdx.x; c < experts * per; c += blockDim.x) {
             const float we = w[c / per];
             float v[8];
-            if (we > 0.f) {
+            if (we != 0.f) {
                 Vec8<T>::load(row + c * 8, v);
 #pragma unroll
                 for (int j = 0; j < 8; ++j) v[j] *= we;
@@ -134,7 +142,7 @@ route_experts_kernel(const float* __restrict__ logits, const T* __restrict__ x, 
     }
     for (int c = threadIdx.x; c < experts * inter; c += blockDim.x) {
         const float we = w[c / inter];
-        row[c] = from_float<T>(we > 0.f ? to_float(row[c]) * we : 0.f);
+        row[c] = from_float<T>(we != 0.f ? to_float(row[c]) * we : 0.f);
     }
 }
 
@@ -142,15 +150,17 @@ route_experts_kernel(const float* __restrict__ logits, const T* __restrict__ x, 
 template <typename T>
 __global__ void __launch_bounds__(kRouteThreads)
 route_topk_kernel(const float* __restrict__ logits, const T* __restrict__ x, const float* __restrict__ router, int width, int experts,
-                  int top, int* __restrict__ ids, float* __restrict__ weights, int mode, float scale) {
-    __shared__ float z[kMaxExperts];
+                  int top, int* __restrict__ ids, float* __restrict__ weights, int mode, float scale, const float* __restrict__ shared_gate,
+                  float* __restrict__ gates) {
+    __shared__ float z[kMaxExperts + 1];
     __shared__ float picked_z[kMaxExperts];
     __shared__ int picked[kMaxExperts];
     pdl_launch();
     pdl_wait();
     const int t = blockIdx.x;
-    router_logits(z, logits, x, router, width, experts, t);
+    router_logits(z, logits, x, router, width, experts, t, shared_gate);
     __syncthreads();
+    if (shared_gate != nullptr && threadIdx.x == 0) gates[t] = 1.f / (1.f + expf(-z[experts]));
     pick_top(z, nullptr, picked, picked_z, experts, top, mode, scale);
     __syncthreads();
     for (int k = threadIdx.x; k < top; k += blockDim.x) {
@@ -216,11 +226,11 @@ gather_picks_kernel(const T* __restrict__ x, int width, const int* __restrict__ 
     }
 }
 
-// out[t] = sum_k weights[t, k] * y[where[t * top + k]] (+ shared[t]) in 32-bit, in the order of k, one rounding.
+// out[t] = sum_k weights[t, k] * y[where[t * top + k]] (+ shared[t], times gates[t] where given) in 32-bit, in the order of k, one rounding.
 template <typename T>
 __global__ void __launch_bounds__(128)
 combine_picks_kernel(const T* __restrict__ y, int width, const int* __restrict__ where, const float* __restrict__ weights, int top,
-                     const T* __restrict__ shared_y, T* __restrict__ out) {
+                     const T* __restrict__ shared_y, const float* __restrict__ gates, T* __restrict__ out) {
     pdl_launch();
     pdl_wait();
     const int t = blockIdx.x;
@@ -234,24 +244,27 @@ combine_picks_kernel(const T* __restrict__ y, int width, const int* __restrict__
             for (int j = 0; j < 8; ++j) acc[j] = fmaf(wk, v[j], acc[j]);
         }
         if (shared_y != nullptr) {
+            const float g = gates != nullptr ? gates[t] : 1.f;
             float v[8];
             Vec8<T>::load(shared_y + (size_t)t * width + c, v);
 #pragma unroll
-            for (int j = 0; j < 8; ++j) acc[j] += v[j];
+            for (int j = 0; j < 8; ++j) acc[j] = fmaf(g, v[j], acc[j]);
         }
         Vec8<T>::store(out + (size_t)t * width + c, acc);
     }
 }
 
 cudaError_t launch_route_topk(int x_dtype, const float* logits, const void* x, const float* router, int width, int n_tokens, int experts,
-                              int top, int* ids, float* weights, cudaStream_t stream, int mode, float scale) {
+                              int top, int* ids, float* weights, cudaStream_t stream, int mode, float scale, const float* shared_gate,
+                              float* gates) {
     if (n_tokens == 0) return cudaSuccess;
     if (experts < 1 || experts > kMaxExperts || top < 1 || top > experts || (x != nullptr && width % 8)) return cudaErrorInvalidValue;
+    if (shared_gate != nullptr && (x == nullptr || gates == nullptr)) return cudaErrorInvalidValue;
     if (x_dtype == kBF16)
         return launch(route_topk_kernel<__nv_bfloat16>, n_tokens, kRouteThreads, 0, stream, logits, (const __nv_bfloat16*)x, router, width,
-                      experts, top, ids, weights, mode, scale);
+                      experts, top, ids, weights, mode, scale, shared_gate, gates);
     return launch(route_topk_kernel<float>, n_tokens, kRouteThreads, 0, stream, logits, (const float*)x, router, width, experts, top, ids,
-                  weights, mode, scale);
+                  weights, mode, scale, shared_gate, gates);
 }
 
 cudaError_t launch_expert_lists(const int* ids, int n_picks, int experts, int list_stride, int* lists, int* counts, cudaStream_t stream) {
@@ -271,25 +284,27 @@ cudaError_t launch_gather_picks(int dtype, const void* x, int width, const int* 
 }
 
 cudaError_t launch_combine_picks(int dtype, const void* y, int width, const int* where, const float* weights, int top, int n_tokens,
-                                 const void* shared_y, void* out, cudaStream_t stream) {
+                                 const void* shared_y, void* out, cudaStream_t stream, const float* gates) {
     if (n_tokens == 0) return cudaSuccess;
     if (width % 8) return cudaErrorInvalidValue;
     if (dtype == kBF16)
         return launch(combine_picks_kernel<__nv_bfloat16>, n_tokens, 128, 0, stream, (const __nv_bfloat16*)y, width, where, weights, top,
-                      (const __nv_bfloat16*)shared_y, (__nv_bfloat16*)out);
+                      (const __nv_bfloat16*)shared_y, gates, (__nv_bfloat16*)out);
     return launch(combine_picks_kernel<float>, n_tokens, 128, 0, stream, (const float*)y, width, where, weights, top,
-                  (const float*)shared_y, (float*)out);
+                  (const float*)shared_y, gates, (float*)out);
 }
 
 cudaError_t launch_route_experts(int dtype, const float* logits, const void* x, const float* router, int width, int n_tokens, int experts,
-                                 int top, void* act, int act_stride, int inter, cudaStream_t stream, int mode, float scale) {
+                                 int top, void* act, int act_stride, int inter, cudaStream_t stream, int mode, float scale,
+                                 const float* shared_gate) {
     if (n_tokens == 0) return cudaSuccess;
+    if (shared_gate != nullptr && x == nullptr) return cudaErrorInvalidValue;
     if (experts < 1 || experts > kMaxExperts || top < 1 || top > experts || (x != nullptr && width % 8)) return cudaErrorInvalidValue;
     if (dtype == kBF16)
         return launch(route_experts_kernel<__nv_bfloat16>, n_tokens, kRouteThreads, 0, stream, logits, (const __nv_bfloat16*)x, router, width,
-                      experts, top, (__nv_bfloat16*)act, act_stride, inter, mode, scale);
+                      experts, top, (__nv_bfloat16*)act, act_stride, inter, mode, scale, shared_gate);
     return launch(route_experts_kernel<float>, n_tokens, kRouteThreads, 0, stream, logits, (const float*)x, router, width, experts, top,
-                  (float*)act, act_stride, inter, mode, scale);
+                  (float*)act, act_stride, inter, mode, scale, shared_gate);
 }
 
 }  // namespace vtb

@@ -25,10 +25,14 @@ template <> __device__ __forceinline__ void store8<float>(float* p, const float*
 // EPI 0: out = sum + bias.  EPI 1 (gate and up rows of w interleaved in runs of 8: g0..g7, u0..u7,
 // g8.., ...): out[token, 8 j + i] = silu(sum of row 16 j + i) * (sum of row 16 j + 8 + i), in 32-bit,
 // silu(z) = z / (1 + exp(-z)) (v1/tensortype/cuda_kernels/silu_product.cu:15-17); out has half the
-// columns.  Every lane of a warp must call it (the swapped form trades values between lanes).
+// columns.  EPI 3: out = max(sum, 0)^2.  Every lane of a warp must call it (the swapped form trades values between lanes).
 template <bool SWAP, int EPI, typename TOut>
 __device__ __forceinline__ void emit16(float (&v)[16], int r, int a_row0, int b_row0, int c0, int rows_a, int rows_b,
                                        const float* __restrict__ bias, TOut* __restrict__ out, int ldo) {
+    if (EPI == 3) {
+#pragma unroll
+        for (int i = 0; i < 16; ++i) v[i] = v[i] > 0.f ? v[i] * v[i] : 0.f;
+    }
     if (SWAP) {
         const int n = a_row0 + r;                  // feature (row of w)
         if (EPI == 1) {

@@ -460,12 +460,17 @@ cudaError_t launch_gemm_tc(int out_dtype, const void* x, const void* w, const fl
                            int* status, cudaStream_t stream, const NextProduct* next) {
     if (m == 0 || n == 0) return cudaSuccess;
     if (k % 8 != 0 || k < 8) return cudaErrorInvalidValue;
-    if (out_dtype == kBF16 && (epilogue == 0 || epilogue == 1) && pair_for(m, n, k))
+    if (out_dtype == kBF16 && (epilogue == 0 || epilogue == 1 || epilogue == 3) && pair_for(m, n, k))
         return launch_gemm_tc_pair(x, w, bias, out, m, n, k, epilogue, 0, scratch, scratch_floats, counters, n_counters, status, stream);
     if (epilogue == 1) {
         if (n % 16 != 0 || bias != nullptr || out_dtype != kBF16) return cudaErrorInvalidValue;
         return launch_typed<1, __nv_bfloat16>(x, w, nullptr, (__nv_bfloat16*)out, m, n, k, scratch, scratch_floats,
                                               counters, n_counters, status, stream, next);
+    }
+    if (epilogue == 3) {
+        if (bias != nullptr || out_dtype != kBF16) return cudaErrorInvalidValue;
+        return launch_typed<3, __nv_bfloat16>(x, w, nullptr, (__nv_bfloat16*)out, m, n, k, scratch, scratch_floats, counters, n_counters,
+                                              status, stream, next);
     }
     if (epilogue == 2) {
         if (out_dtype != kF32 || m > 256) return cudaErrorInvalidValue;

@@ -358,7 +358,7 @@ cudaError_t launch_pair_cfg(const void* x, int m, const void* w, int n, int k, c
 }  // namespace
 
 // bfloat16 out [m, n] (epilogue 0, with bias) or [m, n / 2] (epilogue 1: SiLU(gate) * up over rows of w interleaved
-// in runs of 8).  `bn`: rows of w in a tile: 256, 224 or 192; 0: the one whose rounds of one tile a pair come out best.
+// in runs of 8); epilogue 3: [m, n] of max(sums, 0)^2.  `bn`: rows of w in a tile: 256, 224 or 192; 0: the one whose rounds of one tile a pair come out best.
 cudaError_t launch_gemm_tc_pair(const void* x, const void* w, const float* bias, void* out, int m, int n, int k, int epilogue,
                                 int bn, float* scratch, long long scratch_floats, int* counters, int n_counters, int* status,
                                 cudaStream_t stream) {
@@ -392,6 +392,12 @@ cudaError_t launch_gemm_tc_pair(const void* x, const void* w, const float* bias,
         if (bn == 192) return launch_pair_cfg<192, 7, 1, __nv_bfloat16>(x, m, w, n, k, nullptr, o, n / 2, scratch, scratch_floats, counters, n_counters, status, stream);
         if (bn == 224) return launch_pair_cfg<224, 6, 1, __nv_bfloat16>(x, m, w, n, k, nullptr, o, n / 2, scratch, scratch_floats, counters, n_counters, status, stream);
         return launch_pair_cfg<256, 6, 1, __nv_bfloat16>(x, m, w, n, k, nullptr, o, n / 2, scratch, scratch_floats, counters, n_counters, status, stream);
+    }
+    if (epilogue == 3) {
+        if (bias != nullptr) return cudaErrorInvalidValue;
+        if (bn == 192) return launch_pair_cfg<192, 7, 3, __nv_bfloat16>(x, m, w, n, k, nullptr, o, n, scratch, scratch_floats, counters, n_counters, status, stream);
+        if (bn == 224) return launch_pair_cfg<224, 6, 3, __nv_bfloat16>(x, m, w, n, k, nullptr, o, n, scratch, scratch_floats, counters, n_counters, status, stream);
+        return launch_pair_cfg<256, 6, 3, __nv_bfloat16>(x, m, w, n, k, nullptr, o, n, scratch, scratch_floats, counters, n_counters, status, stream);
     }
     if (epilogue != 0) return cudaErrorInvalidValue;
     if (bn == 192) return launch_pair_cfg<192, 7, 0, __nv_bfloat16>(x, m, w, n, k, bias, o, n, scratch, scratch_floats, counters, n_counters, status, stream);

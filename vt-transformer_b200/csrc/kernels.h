@@ -120,7 +120,7 @@ cudaError_t launch_attention_general(int dtype, const void* y, int stride, int q
 
 // Attention over paged rows that all heads share (attention_latent.cu), bfloat16 on the tensor cores: head h's query
 // [key] at q_col + h * key of q; a row's first v_dim numbers are its value; out[t, out_col + h * v_dim + :].  sinks [heads]
-// or null: exp(sink_h) joins the softmax's denominator.  tiles [n_tiles, 2] (sequence, first token), or null for a step
+// or null: exp(sink_h) joins the softmax's denominator.  window w > 0: a token sees the last w keys up to its own.  tiles [n_tiles, 2] (sequence, first token), or null for a step
 // of single tokens; a tile holds attention_latent_tile_rows() / min(heads, that) tokens.  A step of single tokens may cut every
 // sequence's keys into n_splits (up to 16) runs with a CTA each, merged by a second kernel through part
 // [n_splits, n_tokens, heads, v_dim + 2] float32.
@@ -129,7 +129,7 @@ int attention_latent_tile_rows();
 cudaError_t launch_attention_latent(const void* q, int q_stride, int q_col, void* out, int out_stride, int out_col, const void* pages,
                                     const int* cu_q, const int* q_start, const int* block_table, int table_stride, const int* tiles,
                                     int n_tiles, int n_pages, int heads, int key, int v_dim, int page_size, float scale,
-                                    const float* sinks, int n_splits, float* part, int n_tokens, cudaStream_t stream);
+                                    const float* sinks, int n_splits, float* part, int n_tokens, cudaStream_t stream, int window = 0);
 
 // Differential attention on the tensor cores (attention_diff.cu), bfloat16: the two maps of attention_general with
 // maps 2, for the sizes that attention_diff_supports names.  tiles [n_tiles, 2] (sequence, first token), or null for a
@@ -163,19 +163,22 @@ cudaError_t launch_retention_fix(int dtype, const void* y, int stride, int q_col
 // softmax over the chosen logits weighs them; act[t, e * inter + i] *= weight of e (0 where e was not chosen), for
 // act [n_tokens, act_stride] of `dtype`.
 // The logits are given, or (x not null) formed in the kernel: logits[t, e] = x[t, :] . router[e, :] in 32-bit, x of `dtype`
-// [n_tokens, width], router float [experts, width].
+// [n_tokens, width], router float [experts, width].  shared_gate (float [width], with x): the columns of act behind the experts' are
+// multiplied by sigmoid(x[t, :] . shared_gate); route_topk leaves that number in gates[t], combine_picks multiplies shared_y by it.
 cudaError_t launch_route_experts(int dtype, const float* logits, const void* x, const float* router, int width, int n_tokens, int experts,
-                                 int top, void* act, int act_stride, int inter, cudaStream_t stream, int mode = 0, float scale = 1.f);
+                                 int top, void* act, int act_stride, int inter, cudaStream_t stream, int mode = 0, float scale = 1.f,
+                                 const float* shared_gate = nullptr);
 // The grouped form: ids / weights [n_tokens, top] of each token's picks; lists [experts, list_stride] of the picks (flat
 // index t * top + k) of every expert in rising order and counts [experts]; sorted [n_picks, width] the input rows by
 // expert and where [n_picks] each pick's row; out[t] = sum_k weights[t, k] * y[where[t * top + k]] (+ shared_y[t]).
 cudaError_t launch_route_topk(int x_dtype, const float* logits, const void* x, const float* router, int width, int n_tokens, int experts,
-                              int top, int* ids, float* weights, cudaStream_t stream, int mode = 0, float scale = 1.f);
+                              int top, int* ids, float* weights, cudaStream_t stream, int mode = 0, float scale = 1.f,
+                              const float* shared_gate = nullptr, float* gates = nullptr);
 cudaError_t launch_expert_lists(const int* ids, int n_picks, int experts, int list_stride, int* lists, int* counts, cudaStream_t stream);
 cudaError_t launch_gather_picks(int dtype, const void* x, int width, const int* lists, int list_stride, const int* counts, int experts,
                                 int top, int n_picks, void* sorted, int* where, cudaStream_t stream);
 cudaError_t launch_combine_picks(int dtype, const void* y, int width, const int* where, const float* weights, int top, int n_tokens,
-                                 const void* shared_y, void* out, cudaStream_t stream);
+                                 const void* shared_y, void* out, cudaStream_t stream, const float* gates = nullptr);
 
 // Layers with a latent for each token (latent.cu).
 // Token shift: out[t] = x[t] + (x[t - 1] - x[t]) * mu [width]; before a sequence's first token of the step comes the row
@@ -193,7 +196,7 @@ cudaError_t launch_latent_prepare(int dtype, const void* y, int stride, int q_co
                                   cudaStream_t stream);
 // out[t, out_col + h out_head + j] = sum_i x[t, x_col + h x_head + i] m[h, i, j] (m [heads, inner, outer] of m_dtype), 32-bit sums.
 // mode 1: the `tail` numbers behind a head's inputs are rotated like the shared key part and copied behind its outputs;
-// mode 2: the output is multiplied by sigmoid(gate[t, gate_col + h outer + j]) (gate may be null).
+// mode 2: the output is multiplied by sigmoid(gate[t, gate_col + h outer + j]) (gate may be null); mode 3: by sigmoid(gate[t, gate_col + h]).
 cudaError_t launch_head_matmul(int dtype, int m_dtype, const void* x, int x_stride, int x_col, int x_head, const void* m, int heads,
                                int inner, int outer, void* out, int out_stride, int out_col, int out_head, int n_tokens, int mode,
                                int tail, const float* freq, int half, float mult, const int* positions, const int* token_seq,
@@ -203,6 +206,30 @@ cudaError_t launch_xielu(int dtype, const void* z, void* out, long long n, float
 // out[t, i] = g sigmoid(alpha g) (u + 1), g = min(gate, lim), u = clamp(up, -lim, lim); lim = limit2 from column `split` on.
 cudaError_t launch_gate_clamp(int dtype, const void* gu, void* out, int n_tokens, int inter, int interleave, float alpha, float limit,
                               int split, float limit2, cudaStream_t stream);
+
+// Models whose residual is `streams` streams side by side (streams.cu); x [n_tokens, streams, width] float.
+// Embedding: every stream of x[t] = N(table[id] + second[row]), row = (id before * mul_prev + id * mul_cur) mod buckets, row number
+// `buckets` at position 0; N: root mean square with `weight` (null: none).  state int [state_rows]: a sequence's last token.
+cudaError_t launch_embedding_pair(int dtype, const void* table, const void* second, const int* ids, const int* positions,
+                                  const int* token_seq, const int* cu_q, const int* rows, int n_seqs, int* state, int state_rows,
+                                  const float* weight, float eps, float* x, int streams, int n_tokens, int width, int vocab,
+                                  long long buckets, long long mul_prev, long long mul_cur, int* status, cudaStream_t stream);
+// For r in 0..n_rows: t = rows ? rows[r] : r; with mix [streams, streams] (from, to) and w_out [streams]: x_t <- sum_s mix[s, t] x_s +
+// w_out[t] y, y = delta[t] (of out_dtype) or the sum of parts [n_parts, n_tokens, width], put back if `store`; h = weight * u *
+// rsqrt(mean(u^2) + eps) with u = sum_s w_in[s] x_s.  conv [taps, width] (a step in which every sequence brings one token, or
+// taps == 1): h += sum_j conv[j] h_(t - taps + 1 + j), the rows before from tail [state_rows, taps - 1, width] at
+// seq_rows[token_seq[t]], which moves on by one row.  h goes to out[r] (of out_dtype) or, in 32-bit, to out32[r].
+cudaError_t launch_streams_norm(int out_dtype, float* x, int n_tokens, int streams, int width, const void* delta, const float* parts,
+                                int n_parts, const float* mix, const float* w_out, const float* w_in, const float* weight, float eps,
+                                void* out, float* out32, const int* rows, int n_rows, int store, const float* conv, int taps, float* tail,
+                                int state_rows, const int* token_seq, const int* seq_rows, int n_seqs, int* status, cudaStream_t stream);
+// The same convolution over rows h [tokens, width] of any step: out[t] = h[t] + sum_j w[j] h[t - taps + 1 + j]; tiles [n_tiles, 2]
+// (sequence, first of its new tokens) of per_tile >= taps - 1 tokens; the tail takes the sequence's last taps - 1 rows.
+cudaError_t launch_conv_rows(int out_dtype, const float* h, const float* w, int taps, float* tail, int state_rows, const int* cu_q,
+                             const int* seq_rows, const int* tiles, int n_tiles, int per_tile, void* out, int width, int* status,
+                             cudaStream_t stream);
+// out = max(z, 0)^2, element by element.
+cudaError_t launch_relu_square(int dtype, const void* z, void* out, long long n, cudaStream_t stream);
 
 // dst[t, dst_col + i] = scale * src[t, i] for src [n_tokens, n] and dst [n_tokens, dst_stride], the product in 32-bit.
 // dst[t, dst_col + h v_dim + i] = scale * src[t, h v_dim + i] * sigmoid(y[t, gate_col + (mode 1: h; mode 2: h v_dim + i)]);
@@ -253,6 +280,7 @@ cudaError_t launch_gemm_skinny(int out_dtype, const void* x, const void* w, cons
 // k is not cut.  Launches that share them must not overlap on the GPU.
 // epilogue 0: out[M, N] = sums + bias.  epilogue 1 (bfloat16 out, no bias, N % 16 == 0): the rows of w are
 // gate and up rows interleaved in runs of 8 (g0..g7, u0..u7, g8.., ...) and out[M, N / 2] = silu(gate) * up.
+// epilogue 3 (bfloat16 out, no bias): out = max(sums, 0)^2.
 // epilogue 2 (float out, M <= 256): k is cut into gemm_tc_shares(M, N, K) shares and out[share, M, N] takes each
 // share's sums as they are (the bias with share 0); the kernel that reads them adds them (launch_rmsnorm).
 // NextProduct: the product that the stream runs after this one (its matrix [n, k] of bfloat16, which no kernel writes, and its
@@ -268,7 +296,7 @@ cudaError_t launch_gemm_tc(int out_dtype, const void* x, const void* w, const fl
                            int epilogue, float* scratch, long long scratch_floats, int* counters, int n_counters,
                            int* status, cudaStream_t stream, const NextProduct* next = nullptr);
 // The same product for many rows of x with a tile of 256 rows of x by `bn` (256 or 192) rows of w to a pair of CTAs
-// (tcgen05.mma.cta_group::2): bfloat16 out, epilogue 0 (bias) or 1 (SiLU(gate) * up).
+// (tcgen05.mma.cta_group::2): bfloat16 out, epilogue 0 (bias), 1 (SiLU(gate) * up) or 3 (max(., 0)^2).
 cudaError_t launch_gemm_tc_pair(const void* x, const void* w, const float* bias, void* out, int m, int n, int k, int epilogue,
                                 int bn, float* scratch, long long scratch_floats, int* counters, int n_counters, int* status,
                                 cudaStream_t stream);

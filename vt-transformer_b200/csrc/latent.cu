@@ -171,7 +171,7 @@ constexpr int kHeadCols = 128;       // output columns of a tile, one a thread
 // mode 1 (queries into the latent's space): the `tail` numbers behind a head's `inner` inputs are its rotated part; they
 // are turned by the token's position (pairs (2i, 2i + 1), the first 2 * half of them) and copied behind the head's
 // `outer` outputs.  mode 2 (the latent's result into the head's values): the output is multiplied by
-// sigmoid(gate[t, gate_col + h * outer + j]) where a gate is given.
+// sigmoid(gate[t, gate_col + h * outer + j]) where a gate is given; mode 3: by sigmoid(gate[t, gate_col + h]), one number a head.
 template <typename T, typename TM>
 __global__ void __launch_bounds__(kHeadCols)
 head_matmul_kernel(const T* __restrict__ x, int x_stride, int x_col, int x_head, const TM* __restrict__ m, int inner, int outer,
@@ -206,8 +206,8 @@ head_matmul_kernel(const T* __restrict__ x, int x_stride, int x_col, int x_head,
         for (int tk = 0; tk < kHeadTokens; ++tk) {
             if (tk >= n) break;
             float v = acc[tk];
-            if (mode == 2 && gate != nullptr) {
-                const float z = to_float(gate[(size_t)(t0 + tk) * gate_stride + gate_col + h * outer + j]);
+            if (mode >= 2 && gate != nullptr) {
+                const float z = to_float(gate[(size_t)(t0 + tk) * gate_stride + gate_col + (mode == 3 ? h : h * outer + j)]);
                 v *= 1.f / (1.f + expf(-z));
             }
             out[(size_t)(t0 + tk) * out_stride + out_col + h * out_head + j] = from_float<T>(v);
@@ -296,11 +296,13 @@ head_matmul_mma_kernel(const __nv_bfloat16* __restrict__ x, int x_stride, int x_
         if (tk >= n) continue;
         __nv_bfloat16* op = out + (size_t)(t0 + tk) * out_stride + out_col + (size_t)h * out_head;
         const __nv_bfloat16* gp = (mode == 2 && gate != nullptr) ? gate + (size_t)(t0 + tk) * gate_stride + gate_col + (size_t)h * outer : nullptr;
+        const float of_head = (mode == 3 && gate != nullptr)
+            ? 1.f / (1.f + expf(-__bfloat162float(gate[(size_t)(t0 + tk) * gate_stride + gate_col + h]))) : 1.f;
 #pragma unroll
         for (int nt = 0; nt < kHmCols / 8; ++nt) {
             const int j = n0 + nt * 8 + 2 * tq;
             if (j >= outer) continue;
-            float v0 = acc[nt][2 * i], v1 = acc[nt][2 * i + 1];
+            float v0 = acc[nt][2 * i] * of_head, v1 = acc[nt][2 * i + 1] * of_head;
             if (gp) {
                 v0 *= 1.f / (1.f + expf(-__bfloat162float(gp[j])));
                 v1 *= 1.f / (1.f + expf(-__bfloat162float(gp[j + 1])));

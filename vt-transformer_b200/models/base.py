@@ -6,7 +6,7 @@ from typing import Dict, Optional
 
 import torch
 
-from ..parts.base import CacheView, ParamSpec, ResidualStream, Runtime, build_part
+from ..parts.base import CacheView, ParamSpec, ResidualStream, Runtime, StreamBundle, build_part
 from ..parts.specs import ModelSpec
 from ..weights.loader import WeightSource, check_against, load_report
 
@@ -56,6 +56,17 @@ class DecoderModel:
                     if type(have) is not type(spec) or getattr(have, "kv_heads", None) != getattr(spec, "kv_heads", None) \
                             or getattr(have, "head_dim", None) != getattr(spec, "head_dim", None):
                         raise ValueError(f"run {n}: cache slot {slot} has another layout than block {run.block} reads")
+        need = self.embedding.cache_spec()
+        if need is not None:
+            slot = self.spec.embedding_cache
+            if slot is None or slot in slots:
+                raise ValueError(f"the embedding keeps something of a request and needs a cache slot of its own; the model names {slot}")
+            slots[slot] = need
+        if any(bool(getattr(b, "streams", 0)) != bool(self.spec.streams) or (self.spec.streams and b.streams != self.spec.streams)
+               for b in (*self.spec.blocks, self.spec.embedding)):
+            raise ValueError(f"every block and the embedding of a model of {self.spec.streams} streams must be made for that many")
+        if (self.spec.streams or need is not None) and any(run.add_embedding for run in self.spec.order):
+            raise ValueError("adding the embedding's output again is built for one stream and an embedding that keeps nothing")
         self._slots = slots
 
     def cache_slots(self) -> Dict[int, object]:
@@ -110,7 +121,11 @@ class DecoderModel:
     def forward(self, ctx, views: Dict[int, CacheView]) -> torch.Tensor:
         """Runs the step's tokens and returns float32 logits [wanted rows, vocab].
         ``views[slot]`` is the cache view of a slot for this step."""
-        stream = ResidualStream(self.embedding.forward(ctx), status=ctx.status)
+        if self.spec.embedding_cache is None:
+            x = self.embedding.forward(ctx)
+        else:
+            x = self.embedding.forward(ctx, self._view(views, self.spec.embedding_cache, True))
+        stream = StreamBundle(x, status=ctx.status) if self.spec.streams else ResidualStream(x, status=ctx.status)
         # a run that adds the embedding's output once more reads a second copy of it (the stream itself moves on)
         first = self.embedding.forward(ctx) if any(run.add_embedding for run in self.spec.order) else None
         for run in self.spec.order:

@@ -30,7 +30,7 @@ def _block(cfg: GeponexConfig, i: int, norm: NormSpec) -> BlockSpec:
         mixer = LightningSpec(hidden=cfg.width, heads=m.heads, dim=m.dim, v_dim=m.vdim, decay=m.decay, norm_eps=cfg.norm_eps)
     else:
         mixer = LatentAttentionSpec(hidden=cfg.width, heads=m.heads, head_dim=m.dim, rot_dim=m.rot_dim, v_dim=m.vdim, q_rank=m.q_rank,
-                                    kv_rank=m.kv_rank, scale=m.scale, sink=m.second, gate=m.second, norm_eps=cfg.norm_eps,
+                                    kv_rank=m.kv_rank, scale=m.scale, sink=m.second, gate="element" if m.second else "none", norm_eps=cfg.norm_eps,
                                     position=_position(m.rot))
     f = layer.mlp
     ffn = None

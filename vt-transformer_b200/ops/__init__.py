@@ -391,13 +391,19 @@ _ROUTER_WEIGHTS = {"softmax": 0, "sigmoid_share": 1}
 
 
 def route_topk(logits, top: int, ids: torch.Tensor, weights: torch.Tensor, x=None, router=None, weights_by: str = "softmax",
-               scale: float = 1.0) -> None:
+               scale: float = 1.0, shared_gate=None, gates=None) -> None:
     """ids[t, k] and weights[t, k]: the ``top`` largest router logits of every token in falling order (the lower index
-    among equals) and the softmax over them.  ``logits`` [tokens, experts] float32, or None with the tokens' input rows
+    among equals) and the softmax over them (which is the softmax over all logits, divided by the picks' sum of it), times
+    ``scale``.  ``logits`` [tokens, experts] float32, or None with the tokens' input rows
     ``x`` [tokens, width] and the router's matrix ``router`` [experts, width] (float32), from which the kernel forms
     them as 32-bit dot products.  ``weights_by`` "sigmoid_share": a pick weighs as sigmoid(logit) over the picks' sum of
-    them (+ 1e-20), times ``scale``."""
-    backend().route_topk(logits, int(top), ids, weights, x, router, _ROUTER_WEIGHTS[weights_by], float(scale))
+    them (+ 1e-20), times ``scale``.  ``shared_gate`` [width] float32 (with ``x``): gates[t] = sigmoid(x[t] . shared_gate), in
+    32-bit."""
+    args = (logits, int(top), ids, weights, x, router, _ROUTER_WEIGHTS[weights_by], float(scale))
+    if shared_gate is None:
+        backend().route_topk(*args)
+    else:
+        backend().route_topk(*args, shared_gate, gates)
 
 
 def expert_lists(ids: torch.Tensor, lists: torch.Tensor, counts: torch.Tensor) -> None:
@@ -411,9 +417,13 @@ def gather_picks(x: torch.Tensor, lists: torch.Tensor, counts: torch.Tensor, top
     backend().gather_picks(x, lists, counts, int(top), rows, where)
 
 
-def combine_picks(y: torch.Tensor, where: torch.Tensor, weights: torch.Tensor, shared_y, out: torch.Tensor) -> torch.Tensor:
-    """out[t] = sum_k weights[t, k] * y[where[t * top + k]] (+ shared_y[t]), in 32-bit in the order of k, one rounding."""
-    backend().combine_picks(y, where, weights, shared_y, out)
+def combine_picks(y: torch.Tensor, where: torch.Tensor, weights: torch.Tensor, shared_y, out: torch.Tensor, gates=None) -> torch.Tensor:
+    """out[t] = sum_k weights[t, k] * y[where[t * top + k]] (+ shared_y[t], times gates[t] where given), in 32-bit in the order
+    of k, one rounding."""
+    if gates is None:
+        backend().combine_picks(y, where, weights, shared_y, out)
+    else:
+        backend().combine_picks(y, where, weights, shared_y, out, gates)
     return out
 
 
@@ -445,11 +455,11 @@ LATENT_MAX_RUNS = 16         # the most runs of keys that a sequence is cut into
 
 
 def attention_latent(q, q_col: int, out, out_col: int, pages, ctx, block_table, heads: int, key: int, v_dim: int, scale: float,
-                     sinks=None, status=None):
+                     sinks=None, status=None, window=None):
     """Softmax attention of the step's tokens over paged rows that all heads share: head h's query [key] stands at
     q[t, q_col + h * key + :], a cached token's row of ``pages`` [pages, 1, page_size, key] is every head's key and its first
     ``v_dim`` numbers every head's value; out[t, out_col + h * v_dim + :] = sum_j p_j row_j[:v_dim] with
-    p = softmax_j(scale q . row_j) over the keys j up to the token's position.  ``sinks`` [heads] float32: exp(sinks[h])
+    p = softmax_j(scale q . row_j) over the keys j up to the token's position (``window`` w: over the last w of them).  ``sinks`` [heads] float32: exp(sinks[h])
     joins the denominator (no key, no value, not scaled).  bfloat16 at the sizes the tensor-core kernel takes runs that
     kernel (tiles of 64 rows of (token, head) that share each block of keys; a single token's tile holds its heads, and in a
     step of single tokens every sequence's keys are cut into runs with a CTA each, merged in the order of the runs);
@@ -465,23 +475,30 @@ def attention_latent(q, q_col: int, out, out_col: int, pages, ctx, block_table, 
             # few sequences leave most SMs without a CTA: every sequence's keys are cut into runs, a CTA each
             ctas = ctx.n_seqs * -(-int(heads) // rows)
             runs = min(LATENT_MAX_RUNS, max(1, LATENT_TARGET_CTAS // ctas))
+            if window:          # (no more runs than the window's keys fill with two blocks of 32 each)
+                runs = max(1, min(runs, -(-_key_span(ctx.max_kv_len, int(window), 0) // 64)))
             if runs > 1:
                 part = torch.empty((runs, q.shape[0], int(heads), int(v_dim) + 2), dtype=torch.float32, device=q.device)
         be.attention_latent(q, int(q_col), out, int(out_col), pages, ctx.cu_q, ctx.q_start, block_table, tiles, int(heads), int(key),
-                            int(v_dim), float(scale), sinks, part)
+                            int(v_dim), float(scale), sinks, part, int(window) if window else 0)
         return out
-    return attention_general.__wrapped__(q, q_col, out, out_col, 1.0, pages, pages, ctx, block_table, heads, 1, key, v_dim, None, None,
+    return attention_general.__wrapped__(q, q_col, out, out_col, 1.0, pages, pages, ctx, block_table, heads, 1, key, v_dim, window, None,
                                          scale, status=status, sinks=sinks, values_in_keys=True)
 
 
 def route_experts(logits, top: int, act: torch.Tensor, inter: int, x=None, router=None, weights_by: str = "softmax",
-                  scale: float = 1.0) -> torch.Tensor:
+                  scale: float = 1.0, shared_gate=None) -> torch.Tensor:
     """For every token (row): the ``top`` largest of its router logits [experts] (float32; the lower index among
     equals) choose its experts, the softmax over the chosen logits weighs them; columns [e * inter, (e + 1) * inter) of
     ``act`` (what expert e's last product multiplies) are multiplied by expert e's weight, and set to zero for an
     expert that was not chosen.  Columns beyond experts * inter (an expert that every token uses) stay.  ``logits`` may be
-    None with ``x`` and ``router`` given, and ``weights_by`` and ``scale``, as for ``route_topk``."""
-    backend().route_experts(logits, int(top), act, int(inter), x, router, _ROUTER_WEIGHTS[weights_by], float(scale))
+    None with ``x`` and ``router`` given, and ``weights_by`` and ``scale``, as for ``route_topk``.  ``shared_gate`` [width]
+    float32 (with ``x``): the columns beyond are multiplied by sigmoid(x[t] . shared_gate), formed in 32-bit."""
+    args = (logits, int(top), act, int(inter), x, router, _ROUTER_WEIGHTS[weights_by], float(scale))
+    if shared_gate is None:
+        backend().route_experts(*args)
+    else:
+        backend().route_experts(*args, shared_gate)
     return act
 
 
@@ -509,8 +526,8 @@ def head_matmul(x, x_col: int, x_head: int, m, out, out_col: int, out_head: int,
     """out[t, out_col + h * out_head + j] = sum_i x[t, x_col + h * x_head + i] * m[h, i, j] for m [heads, inner, outer], the
     sums in 32-bit in the order of i.  ``mode`` "rotated_tail": the ``tail`` numbers behind a head's inputs are rotated
     like ``latent_prepare``'s shared key part and copied behind the head's outputs; "gate": the result is multiplied by
-    sigmoid(gate[t, gate_col + h * outer + j]) where ``gate`` is given."""
-    code = {"plain": 0, "rotated_tail": 1, "gate": 2}[mode]
+    sigmoid(gate[t, gate_col + h * outer + j]) where ``gate`` is given; "head_gate": by sigmoid(gate[t, gate_col + h])."""
+    code = {"plain": 0, "rotated_tail": 1, "gate": 2, "head_gate": 3}[mode]
     backend().head_matmul(x, int(x_col), int(x_head), m, out, int(out_col), int(out_head), code, int(tail), frequencies,
                           float(mult), None if ctx is None else ctx.positions, None if ctx is None else ctx.token_seq, gate,
                           int(gate_col))
@@ -530,6 +547,83 @@ def gate_clamp(gu: torch.Tensor, out: torch.Tensor, interleave: int, alpha: floa
     n = out.shape[1]
     backend().gate_clamp(gu, out, int(interleave), float(alpha), float(limit), int(split) if limit2 is not None else n,
                          float(limit if limit2 is None else limit2))
+    return out
+
+
+def relu_square(z: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """out = max(z, 0)^2 element by element, in 32-bit with one rounding; ``out`` may be ``z``."""
+    backend().relu_square(z, out)
+    return out
+
+
+def linear_relu_square(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, status=None, then=None) -> torch.Tensor:
+    """out[T, N] = max(x w^T, 0)^2.  bfloat16: one tcgen05 kernel whose epilogue squares the 32-bit sums.  Otherwise the
+    product and the elementwise kernel."""
+    be = backend()
+    if x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and not (x.shape[0] <= SKINNY_MAX_ROWS and SMALL_BATCH_KERNEL == "skinny"):
+        scratch, counters = _split_workspace(x.device)
+        global launches
+        launches += 1
+        be.gemm_tc(x, w, None, out, status, scratch, counters, 3, **_ahead(then))
+        return out
+    linear(x, w, None, out, status)
+    return relu_square(out, out)
+
+
+def embedding_pair(table: torch.Tensor, second: torch.Tensor, ctx, state: torch.Tensor, x: torch.Tensor, mul_prev: int, mul_cur: int,
+                   weight=None, eps: float = 0.0, status=None) -> torch.Tensor:
+    """Every stream of x [T, streams, width] (float32) = N(table[id] + second[row]) with row = (id of the token before * mul_prev +
+    id * mul_cur) mod (rows of ``second`` - 1) and the last row for a sequence's first token.  N: divided by the root mean
+    square and multiplied by ``weight`` (None: nothing).  ``state`` int32, a number a request row: the request's last
+    token, read for the step's first token of a sequence and renewed.  Rows of padding tokens become zero."""
+    backend().embedding_pair(table, second, ctx.token_ids, ctx.positions, ctx.token_seq, ctx.cu_q, ctx.rows, state, weight, float(eps), x,
+                             int(mul_prev), int(mul_cur), status)
+    return x
+
+
+CONV_FUSED_MAX_WIDTH = 6144      # widest rows whose convolution the kernel of a step of single tokens takes along
+CONV_TILE = 16                   # tokens that a CTA of the convolution over a step's rows walks
+
+
+def streams_norm(x: torch.Tensor, w_in: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, change=None, rows=None,
+                 store: bool = True, conv=None, tail=None, ctx=None, status=None) -> torch.Tensor:
+    """From one sublayer to the next over a residual of several streams, x [T, streams, width] (float32).  ``change`` =
+    (y, mix [streams, streams], w_out [streams]): x_t <- sum_s mix[s, t] x_s + w_out[t] y first, with y a tensor [T, width] of
+    out's dtype or a ``SplitSum``, put back into x if ``store``.  Then out = weight * u / sqrt(mean(u^2) + eps) with
+    u = sum_s w_in[s] x_s over the rows ``rows`` (all).  With ``conv`` [taps, width] (the last tap the present row's) out
+    is h_t + sum_j conv[j] h_(t - taps + 1 + j) of the normed rows h (before their rounding): the rows before a
+    sequence's first token of the step come from ``tail`` [request rows, taps - 1, width] (float32, oldest first, zeros at
+    admission), which is renewed.  In a step of single tokens that is the same kernel; otherwise the normed rows go
+    through memory in 32-bit and a second kernel convolves them.  All in 32-bit, one rounding."""
+    global launches
+    be = backend()
+    y, mix, w_out = change if change is not None else (None, None, None)
+    if isinstance(y, SplitSum):
+        y = y.shares
+    common = dict(status=status)
+    if conv is None:
+        be.streams_norm(x, y, mix, w_out, w_in, weight, float(eps), out, rows, bool(store), **common)
+        return out
+    taps, width = conv.shape
+    singles = ctx.max_q_len == 1 and ctx.n_tokens == ctx.n_seqs
+    if taps == 1 or (singles and width <= CONV_FUSED_MAX_WIDTH):
+        be.streams_norm(x, y, mix, w_out, w_in, weight, float(eps), out, None, bool(store), conv=conv, tail=tail,
+                        token_seq=ctx.token_seq, seq_rows=ctx.rows, **common)
+        return out
+    h = torch.empty(out.shape, dtype=torch.float32, device=out.device)
+    be.streams_norm(x, y, mix, w_out, w_in, weight, float(eps), h, None, bool(store), wide=True,
+                    dtype_of_delta=1 if out.dtype == torch.bfloat16 else 0, **common)
+    launches += 1
+    per_tile = max(CONV_TILE, taps - 1)
+    if singles:
+        tiles = ctx.extras.get("conv_single_tiles")
+        if tiles is None:
+            tiles = torch.zeros((ctx.n_seqs, 2), dtype=torch.int32, device=out.device)
+            tiles[:, 0] = torch.arange(ctx.n_seqs, dtype=torch.int32, device=out.device)
+            ctx.extras["conv_single_tiles"] = tiles
+    else:
+        tiles = _attention_tiles(ctx, per_tile, out.device)
+    be.conv_rows(h, conv, tail, ctx.cu_q, ctx.rows, tiles, per_tile, out, status)
     return out
 
 
@@ -1022,6 +1116,6 @@ def _counted(fn):
     return wrapper
 
 
-for _name in ("gate_into", "gated_delta_scan", "conv_tail_update", "memory_scan", "normed_sum", "add_rows", "embedding", "logits_scale_cap", "rmsnorm", "layernorm", "polynorm", "scale_into", "head_norm_gate", "gla_scan", "delta_scan", "retention_scan", "route_experts", "attention_differential", "route_topk", "expert_lists", "gather_picks", "combine_picks",
+for _name in ("embedding_pair", "streams_norm", "relu_square", "gate_into", "gated_delta_scan", "conv_tail_update", "memory_scan", "normed_sum", "add_rows", "embedding", "logits_scale_cap", "rmsnorm", "layernorm", "polynorm", "scale_into", "head_norm_gate", "gla_scan", "delta_scan", "retention_scan", "route_experts", "attention_differential", "route_topk", "expert_lists", "gather_picks", "combine_picks",
               "token_shift", "latent_prepare", "head_matmul", "attention_latent", "xielu", "gate_clamp", "attention_prepare", "attention_general", "silu_mul", "rope_store", "linear", "paged_attention", "argmax", "sample"):  # the others count where they launch
     globals()[_name] = _counted(globals()[_name])

@@ -114,8 +114,9 @@ class KVCacheSpec:
 @dataclass(frozen=True)
 class LatentCacheSpec:
     """One row of ``width`` numbers for each token, in pages (a latent from which a layer makes every head's keys and
-    values, with a key part that the heads share behind it); all tokens are kept."""
+    values, with a key part that the heads share behind it); ``window`` None keeps all tokens, w the last w."""
     width: int
+    window: Optional[int] = None
 
 
 @dataclass(frozen=True)
@@ -168,7 +169,7 @@ def cache_layout(spec):
 register_cache_kind(KVCacheSpec, lambda s: PagedLayout((("k", s.kv_heads * s.k_maps, s.head_dim),
                                                         ("v", s.kv_heads, s.v_dim if s.v_dim else s.head_dim)), s.window,
                                                        s.keep_first if s.window is not None else 0))
-register_cache_kind(LatentCacheSpec, lambda s: PagedLayout((("c", 1, s.width),), None, 0))
+register_cache_kind(LatentCacheSpec, lambda s: PagedLayout((("c", 1, s.width),), s.window, 0))
 register_cache_kind(StateSpec, lambda s: StateLayout(tuple(s.shape), s.dtype))
 
 
@@ -233,6 +234,10 @@ class Norm(Part):
     x, and normed.  With ``rows`` (int32 indices) only those rows are done, packed in that order.
     Returns the normed rows in the compute dtype.
 
+    ``over_streams(stream, w_in, rows=None, store=True, conv=None, tail=None, ctx=None)`` (a norm that sets ``takes_streams``):
+    the norm of sum_s w_in[s] x_s (``w_in`` None: of the sum) over the streams of a ``StreamBundle``, with the change that is pending there applied on
+    the way, and with the short convolution over the normed rows where one is given (``ops.streams_norm``).
+
     A norm whose kernel can add the unadded 32-bit shares of a matrix product itself sets ``takes_shares``; it is
     then given what ``ops.linear_to_stream`` returned as it is.  Any other norm gets an ordinary tensor.
 
@@ -243,11 +248,15 @@ class Norm(Part):
     category = "norm"
     takes_shares = False
     takes_post = False
+    takes_streams = False
 
     def __call__(self, x, delta=None, rows=None, status=None, post=None):
         raise NotImplementedError
 
     def weighted(self):
+        raise NotImplementedError
+
+    def over_streams(self, stream, w_in, rows=None, store=True, conv=None, tail=None, ctx=None):
         raise NotImplementedError
 
 
@@ -295,11 +304,16 @@ class Block(Part):
 
 
 class Embedding(Part):
-    """``forward(ctx) -> x``: the step's token ids (``ctx.token_ids``, -1 for padding) as the 32-bit residual
-    stream [T, hidden].  ``prefix`` is the tensor's full name.  ``step_bytes(n_tokens)``: bytes it reads a step."""
+    """``forward(ctx, cache=None) -> x``: the step's token ids (``ctx.token_ids``, -1 for padding) as the 32-bit residual
+    stream [T, hidden], or [T, streams, hidden] in a model of several streams.  ``prefix`` is the tensor's full name.
+    ``step_bytes(n_tokens)``: bytes it reads a step.  ``cache_spec()``: what it keeps of a request between steps (None or one
+    spec); ``forward`` then gets the view of it."""
     category = "embedding"
 
-    def forward(self, ctx):
+    def cache_spec(self):
+        return None
+
+    def forward(self, ctx, cache=None):
         raise NotImplementedError
 
     def step_bytes(self, n_tokens: int) -> int:
@@ -346,6 +360,36 @@ class ResidualStream:
         if self.pending is not None:
             raise RuntimeError("the residual stream holds a delta that no norm has added yet")
         self.pending, self.pending_post = delta, post
+
+
+class StreamBundle:
+    """A residual of several 32-bit streams [T, streams, H] and a sublayer's result not yet given to them.
+
+    A block leaves (y, mix [streams, streams], w_out [streams]) in ``pending``: x_t <- sum_s mix[s, t] x_s + w_out[t] y for
+    all streams at once.  The norm that prepares the next sublayer applies it while it reads the streams
+    (``Norm.over_streams``), so they are read and written once a sublayer.  ``normed`` is what the head asks for: the norm
+    of the streams' sum."""
+
+    def __init__(self, x: torch.Tensor, status: Optional[torch.Tensor] = None):
+        if x.dim() != 3:
+            raise ValueError("a bundle of streams is [tokens, streams, hidden]: the embedding must make every stream")
+        self.x = x
+        self.status = status
+        self.pending = None
+
+    def take(self):
+        change, self.pending = self.pending, None
+        return change
+
+    def add(self, y, mix, w_out) -> None:
+        if self.pending is not None:
+            raise RuntimeError("the streams hold a result that no norm has given to them yet")
+        self.pending = (y, mix, w_out)
+
+    def normed(self, norm: Norm, rows=None):
+        if not getattr(norm, "takes_streams", False):
+            raise RuntimeError(f"norm '{norm.spec.kind}' cannot read several streams")
+        return norm.over_streams(self, None, rows=rows, store=False)
 
 
 # ----------------------------------------------------------------------------- registry

@@ -88,6 +88,87 @@ class SandwichBlock(PreNormBlock):
         stream.add(self.ffn.forward(h, ctx), post=(self.post2.weighted(), s.post2.eps, s.residual_mult))
 
 
+def _register_stream_initialisers():
+    """Starts of the random-weights mode under which several streams keep the size of one: a sublayer reads about the mean
+    of the streams, writes about as much as it returns into each, and the streams stay mostly themselves."""
+    from ..weights.loader import register_initialiser
+    noise = lambda shape, g, device: torch.randn(shape, generator=g, dtype=torch.float32, device=device)
+    register_initialiser("stream_in", lambda shape, g, sigma, device: (1.0 + 0.2 * noise(shape, g, device)) / shape[0], replace=True)
+    register_initialiser("stream_out", lambda shape, g, sigma, device: 1.0 + 0.2 * noise(shape, g, device), replace=True)
+    register_initialiser("stream_mix", lambda shape, g, sigma, device: torch.eye(shape[0], dtype=torch.float32, device=device)
+                         + 0.1 * noise(shape, g, device) / shape[0], replace=True)
+
+
+_register_stream_initialisers()
+
+
+@register_part("block", "streams")
+class StreamsBlock(PreNormBlock):
+    """A layer of a model whose residual is several streams (``BlockSpec``, ``streams``): for each of its two sublayers one
+    kernel gives the streams the result of the sublayer before, reads them as one vector, norms it and (in steps of single
+    tokens) convolves it with the rows before; then the sublayer, whose result waits for the next such kernel.  The
+    first of the run's cache slots are the convolutions' rows, one slot a sublayer, then what the mixer keeps."""
+
+    def __init__(self, spec, prefix, rt):
+        super().__init__(spec, prefix, rt)
+        if not 1 <= spec.streams <= 16:
+            raise ValueError(f"streams block: {spec.streams} streams; 1 to 16 are built")
+        if not 0 <= spec.conv_taps <= 16:
+            raise ValueError(f"streams block: a convolution of {spec.conv_taps} taps; up to 16 are built")
+        for n in (self.norm1, self.norm2):
+            if n is not None and not getattr(n, "takes_streams", False):
+                raise ValueError(f"streams block: norm '{n.spec.kind}' cannot read several streams")
+        self.sublayers = 1 if self.ffn is None else 2
+
+    def _kept_rows(self) -> int:
+        return self.sublayers if self.spec.conv_taps > 1 else 0
+
+    def cache_spec(self):
+        inner = self.mixer.cache_spec()
+        kept = () if inner is None else (tuple(inner) if isinstance(inner, (tuple, list)) else (inner,))
+        rows = StateSpec((self.spec.conv_taps - 1, self.spec.norm1.size), torch.float32)
+        kept = (rows,) * self._kept_rows() + kept
+        return None if not kept else (kept[0] if len(kept) == 1 else kept)
+
+    def param_specs(self):
+        s, out = self.spec, super().param_specs()
+        for q in range(self.sublayers):
+            p = self.prefix + s.stream_prefixes[q]
+            for name, shape, init in zip(s.stream_names, ((s.streams,), (s.streams,), (s.streams, s.streams)),
+                                         ("stream_in", "stream_out", "stream_mix")):
+                out[p + name] = ParamSpec(shape, role="vector", init=init)
+            if s.conv_taps:
+                out[self.prefix + s.conv_names[q]] = ParamSpec((s.norm1.size, s.conv_taps), role="vector", init="conv_taps")
+        return out
+
+    def load(self, get) -> None:
+        super().load(get)
+        s, rt = self.spec, self.rt
+        self.read, self.write, self.mix, self.conv = [], [], [], []
+        for q in range(self.sublayers):
+            p = self.prefix + s.stream_prefixes[q]
+            for kept, name in zip((self.read, self.write, self.mix), s.stream_names):
+                kept.append(rt.param(get(p + name), "vector"))
+            # a tap's weights side by side, as the kernels read them
+            self.conv.append(rt.param(get(self.prefix + s.conv_names[q]), "vector").t().contiguous() if s.conv_taps else None)
+
+    def weight_bytes(self) -> int:
+        small = [t for kept in (self.read, self.write, self.mix, self.conv) for t in kept if t is not None]
+        return super().weight_bytes() + sum(t.numel() * t.element_size() for t in small)
+
+    def forward(self, stream, ctx, cache):
+        views = list(cache) if isinstance(cache, (tuple, list)) else ([] if cache is None else [cache])
+        n = self._kept_rows()
+        tails, rest = [v.state for v in views[:n]] or [None] * self.sublayers, tuple(views[n:])
+        h = self.norm1.over_streams(stream, self.read[0], conv=self.conv[0], tail=tails[0], ctx=ctx)
+        y = self.mixer.forward(h, ctx, None if not rest else (rest[0] if len(rest) == 1 else rest))
+        stream.add(y, self.mix[0], self.write[0])
+        if self.ffn is None:
+            return
+        h = self.norm2.over_streams(stream, self.read[1], conv=self.conv[1], tail=tails[1], ctx=ctx)
+        stream.add(self.ffn.forward(h, ctx), self.mix[1], self.write[1])
+
+
 @register_part("block", "postnorm")
 class PostNormBlock(Block):
     """x <- norm1(a x + mixer(shift(x))); x <- norm2(a x + ffn(x)): the norms come after the sums and their result is the

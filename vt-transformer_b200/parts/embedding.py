@@ -3,7 +3,7 @@ from __future__ import annotations
 
 import torch
 
-from .base import Embedding, Head, ParamSpec, build_part, register_part
+from .base import Embedding, Head, ParamSpec, StateSpec, build_part, register_part
 
 
 @register_part("embedding", "table")
@@ -22,10 +22,56 @@ class TableEmbedding(Embedding):
     def step_bytes(self, n_tokens: int) -> int:
         return n_tokens * self.spec.hidden * self.table.element_size()
 
-    def forward(self, ctx):
+    def forward(self, ctx, cache=None):
         x = torch.empty((ctx.n_tokens, self.spec.hidden), dtype=torch.float32, device=self.rt.device)
         self.rt.ops.embedding(self.table, ctx.token_ids, x, status=ctx.status, scale=self.spec.scale)
         return x
+
+
+@register_part("embedding", "pair")
+class PairEmbedding(Embedding):
+    """See ``EmbeddingSpec``: a token's row plus a row of a second table that the pair (token before, token) picks, normed
+    where a norm is given, in every stream of the residual; one kernel.  A request keeps its last token (a state slot)."""
+
+    graph_safe = True
+
+    def __init__(self, spec, prefix, rt):
+        super().__init__(spec, prefix, rt)
+        if spec.pair is None:
+            raise ValueError("pair embedding: 'pair' = (buckets, factor of the token before, factor of the token)")
+        if spec.scale != 1.0:
+            raise ValueError("pair embedding: a scale is not built")
+        if spec.norm is not None and (spec.norm.kind != "rmsnorm" or spec.norm.groups != 1):
+            raise ValueError("pair embedding: its norm is a root-mean-square norm without groups")
+        self.norm = build_part("norm", spec.norm, spec.norm_name, rt) if spec.norm is not None else None
+
+    def cache_spec(self):
+        return StateSpec((1,), torch.int32)
+
+    def param_specs(self):
+        s = self.spec
+        out = {self.prefix: ParamSpec((s.vocab, s.hidden)), s.pair_name: ParamSpec((s.pair[0] + 1, s.hidden))}
+        if self.norm is not None:
+            out.update(self.norm.param_specs())
+        return out
+
+    def load(self, get) -> None:
+        self.table, self.second = self.rt.load(get, self.prefix), self.rt.load(get, self.spec.pair_name)
+        if self.table.dtype != self.second.dtype:
+            self.table, self.second = self.table.float(), self.second.float()
+        if self.norm is not None:
+            self.norm.load(get)
+
+    def step_bytes(self, n_tokens: int) -> int:
+        return 2 * n_tokens * self.spec.hidden * self.table.element_size()
+
+    def forward(self, ctx, cache=None):
+        s = self.spec
+        x = torch.empty((ctx.n_tokens, max(1, s.streams), s.hidden), dtype=torch.float32, device=self.rt.device)
+        weight, eps = (None, 0.0) if self.norm is None else (self.norm.weighted(), s.norm.eps)
+        self.rt.ops.embedding_pair(self.table, self.second, ctx, cache.state, x, s.pair[1], s.pair[2], weight=weight, eps=eps,
+                                   status=ctx.status)
+        return x if s.streams else x.view(ctx.n_tokens, s.hidden)
 
 
 @register_part("head", "linear")

@@ -7,6 +7,9 @@ from .base import LatentCacheSpec, ParamSpec, build_part, register_part
 from .projected import ProjectedMixer, _round_up, pack_rows
 
 
+_GATE_MODES = {"none": "plain", "element": "gate", "head": "head_gate"}
+
+
 @register_part("mixer", "latent_attention")
 class LatentAttention(ProjectedMixer):
     """See ``LatentAttentionSpec``.  A token keeps its normed latent c and the rotated key part r that the heads share,
@@ -25,12 +28,14 @@ class LatentAttention(ProjectedMixer):
         if pos.kind != "none" and (pos.dim % 2 or pos.dim > spec.rot_dim):
             raise ValueError(f"latent attention: the rotation covers {pos.dim} dimensions; it must be even and at most the "
                              f"rotated part's {spec.rot_dim}")
+        if spec.gate not in ("none", "element", "head"):
+            raise ValueError(f"latent attention: gate '{spec.gate}' is not built; known: none, element, head")
         self.position = build_part("position", pos, prefix, rt)
         self.q_head = spec.head_dim + spec.rot_dim            # a head's query as the up projection leaves it
         self.key = spec.kv_rank + spec.rot_dim                # a token's row, and a head's query in the latent's space
 
     def cache_spec(self):
-        return LatentCacheSpec(self.key)
+        return LatentCacheSpec(self.key, self.spec.window)
 
     def param_specs(self):
         s, p = self.spec, self.prefix
@@ -44,14 +49,14 @@ class LatentAttention(ProjectedMixer):
         }
         if s.sink:
             out[p + sink] = ParamSpec((s.heads,), role="vector")
-        if s.gate:
-            out[p + g] = ParamSpec((s.heads * s.v_dim, s.hidden))
+        if s.gate != "none":
+            out[p + g] = ParamSpec((s.heads if s.gate == "head" else s.heads * s.v_dim, s.hidden))
         return out
 
     def load(self, get) -> None:
         s, p, rt = self.spec, self.prefix, self.rt
         dq, dqn, uq, dkv, dkvn, uk, uv, o, sink, g = s.names
-        self._in = [rt.param(get(p + n)) for n in ((dq, dkv, g) if s.gate else (dq, dkv))]
+        self._in = [rt.param(get(p + n)) for n in ((dq, dkv, g) if s.gate != "none" else (dq, dkv))]
         self.w_o = rt.param(get(p + o))
         self.q_weight = rt.param(get(p + dqn), "vector")
         self.k_weight = rt.param(get(p + dkvn), "vector")
@@ -101,10 +106,10 @@ class LatentAttention(ProjectedMixer):
                         ctx=ctx)
         oc = torch.empty((T, s.heads * s.kv_rank), dtype=y.dtype, device=dev)
         ops.attention_latent(qa, 0, oc, 0, pages, ctx, cache.block_table, s.heads, self.key, s.kv_rank, s.scale, sinks=self.sinks,
-                             status=ctx.status)
+                             status=ctx.status, window=s.window)
         direct = out_scale == 1.0
         o = out if direct else torch.empty((T, s.heads * s.v_dim), dtype=y.dtype, device=dev)
-        ops.head_matmul(oc, 0, s.kv_rank, self.v, o, out_col if direct else 0, s.v_dim, mode="gate" if s.gate else "plain",
-                        gate=y if s.gate else None, gate_col=cols[2] if s.gate else 0)
+        ops.head_matmul(oc, 0, s.kv_rank, self.v, o, out_col if direct else 0, s.v_dim, mode=_GATE_MODES[s.gate],
+                        gate=y if s.gate != "none" else None, gate_col=cols[2] if s.gate != "none" else 0)
         if not direct:
             ops.scale_into(o, out, out_col, out_scale)

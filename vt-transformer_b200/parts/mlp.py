@@ -146,7 +146,8 @@ class XieluMLP(FeedForward):
 
 @register_part("feed_forward", "experts")
 class Experts(FeedForward):
-    """See ``ExpertsSpec``.  The router's logits are 32-bit dot products formed inside the routing kernel (its matrix is
+    """See ``ExpertsSpec`` (the description below is that of gated experts; without a gate matrix the packed matrix holds the up
+    matrices alone).  The router's logits are 32-bit dot products formed inside the routing kernel (its matrix is
     kept in 32-bit).  All experts'
     gate and up matrices, and the shared expert's, are one packed matrix, so silu(gate) * up of every expert for every
     token is ONE product with the activation in its epilogue; one kernel then picks each token's experts, forms their
@@ -165,15 +166,22 @@ class Experts(FeedForward):
 
     def __init__(self, spec, prefix, rt):
         super().__init__(spec, prefix, rt)
-        if spec.activation not in ("silu", "clamped"):
-            raise ValueError(f"experts: activation '{spec.activation}' is not built; known: silu, clamped")
+        if spec.activation not in ("silu", "clamped", "relu_square"):
+            raise ValueError(f"experts: activation '{spec.activation}' is not built; known: silu, clamped, relu_square")
+        if spec.shared_gate_name is not None and not spec.shared_inter:
+            raise ValueError("experts: a shared expert's gate without a shared expert")
+        self.gated = spec.activation != "relu_square"          # the experts have a gate matrix beside the up matrix
+        self.shared_gate = None
         if spec.router_weights not in ("softmax", "sigmoid_share"):
             raise ValueError(f"experts: router weights '{spec.router_weights}' are not built; known: softmax, sigmoid_share")
 
     def gate_up(self, x, w_gate_up, act, limit: float, then=None, split: int = 0, limit2=None):
         """act = what the last product multiplies, from x and the interleaved gate and up matrices: silu(gate) * up in the
-        product's epilogue, or, for the clamped form, the product and then the activation's kernel."""
+        product's epilogue, or, for the clamped form, the product and then the activation's kernel; without a gate matrix
+        the square of relu in the epilogue of the product with the up matrix."""
         s, ops = self.spec, self.rt.ops
+        if not self.gated:
+            return ops.linear_relu_square(x, w_gate_up, act, then=then)
         if s.activation == "silu":
             return ops.linear_silu_mul(x, w_gate_up, act, then=then)
         gu = torch.empty((x.shape[0], w_gate_up.shape[0]), dtype=x.dtype, device=x.device)
@@ -188,9 +196,12 @@ class Experts(FeedForward):
         if s.shared_inter:
             blocks.append((p + s.shared_prefix, s.shared_inter))
         for prefix, inter in blocks:
-            out[prefix + g] = ParamSpec((inter, s.hidden))
+            if self.gated:
+                out[prefix + g] = ParamSpec((inter, s.hidden))
             out[prefix + u] = ParamSpec((inter, s.hidden))
             out[prefix + d] = ParamSpec((s.hidden, inter))
+        if s.shared_gate_name is not None:
+            out[p + s.shared_gate_name] = ParamSpec((1, s.hidden))
         return out
 
     def load(self, get) -> None:
@@ -203,16 +214,18 @@ class Experts(FeedForward):
             blocks.append((p + s.shared_prefix, s.shared_inter, -(-s.shared_inter // 8) * 8))
         gate_up, down = [], []
         for prefix, inter, padded in blocks:
-            mats = [rt.param(get(prefix + n)) for n in (g, u, d)]
+            mats = [rt.param(get(prefix + n)) for n in ((g, u, d) if self.gated else (u, d))]
             if len({m.dtype for m in mats}) > 1:
                 mats = [m.float() for m in mats]
-            wg, wu, wd = mats
+            wd = mats.pop()
             if padded != inter:
-                zeros = torch.zeros((padded - inter, s.hidden), dtype=wg.dtype, device=wg.device)
-                wg, wu = torch.cat([wg, zeros]), torch.cat([wu, zeros])
+                zeros = torch.zeros((padded - inter, s.hidden), dtype=wd.dtype, device=wd.device)
+                mats = [torch.cat([m, zeros]) for m in mats]
                 wd = torch.cat([wd, torch.zeros((s.hidden, padded - inter), dtype=wd.dtype, device=wd.device)], dim=1)
-            gate_up.append(rt.ops.interleave_gate_up(wg, wu))
+            gate_up.append(rt.ops.interleave_gate_up(*mats) if self.gated else mats[0])
             down.append(wd)
+        if s.shared_gate_name is not None:
+            self.shared_gate = rt.param(get(p + s.shared_gate_name), "vector").view(-1)
         if len({m.dtype for m in gate_up + down}) > 1:
             gate_up, down = [m.float() for m in gate_up], [m.float() for m in down]
         self.w_gate_up = torch.cat(gate_up, dim=0).contiguous()
@@ -225,10 +238,11 @@ class Experts(FeedForward):
         self.down_of = [d.contiguous() for d in down]
 
     def weight_bytes(self) -> int:
-        return sum(m.numel() * m.element_size() for m in (self.router, self.w_gate_up, self.w_down))
+        mats = (self.router, self.w_gate_up, self.w_down, self.shared_gate)
+        return sum(m.numel() * m.element_size() for m in mats if m is not None)
 
     def first_product(self):
-        return self.rt.ops.product_hint(self.w_gate_up, "silu_mul")
+        return self.rt.ops.product_hint(self.w_gate_up, "silu_mul" if self.gated else "linear")
 
     def forward(self, h, ctx):
         s, ops = self.spec, self.rt.ops
@@ -238,8 +252,9 @@ class Experts(FeedForward):
         act = torch.empty((T, self.w_down.shape[1]), dtype=h.dtype, device=h.device)
         self.gate_up(h, self.w_gate_up, act, s.limit, then=ops.product_hint(self.w_down, "stream"),
                      split=s.experts * self.inter, limit2=s.shared_limit if s.shared_inter else None)
-        # the router's logits are formed there, in 32-bit
-        ops.route_experts(None, s.top, act, self.inter, x=h, router=self.router, weights_by=s.router_weights, scale=s.router_scale)
+        # the router's logits are formed there, in 32-bit (and the shared expert's gate)
+        ops.route_experts(None, s.top, act, self.inter, x=h, router=self.router, weights_by=s.router_weights, scale=s.router_scale,
+                          shared_gate=self.shared_gate)
         return ops.linear_to_stream(act, self.w_down, None, then=self.then)
 
     def grouped(self, h):
@@ -248,7 +263,9 @@ class Experts(FeedForward):
         T, picks = h.shape[0], h.shape[0] * s.top
         ids = torch.empty((T, s.top), dtype=torch.int32, device=dev)
         weights = torch.empty((T, s.top), dtype=torch.float32, device=dev)
-        ops.route_topk(None, s.top, ids, weights, x=h, router=self.router, weights_by=s.router_weights, scale=s.router_scale)
+        gates = None if self.shared_gate is None else torch.empty((T,), dtype=torch.float32, device=dev)
+        ops.route_topk(None, s.top, ids, weights, x=h, router=self.router, weights_by=s.router_weights, scale=s.router_scale,
+                       shared_gate=self.shared_gate, gates=gates)
         lists = torch.empty((s.experts, T), dtype=torch.int32, device=dev)
         counts = torch.empty((s.experts,), dtype=torch.int32, device=dev)
         ops.expert_lists(ids, lists, counts)
@@ -270,4 +287,4 @@ class Experts(FeedForward):
                 ops.linear(act[at:at + n], self.down_of[e], None, y[at:at + n])
             at += n
         out = torch.empty((T, s.hidden), dtype=h.dtype, device=dev)
-        return ops.combine_picks(y, where, weights, shared_y, out)
+        return ops.combine_picks(y, where, weights, shared_y, out, gates=gates)

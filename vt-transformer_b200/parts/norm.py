@@ -14,8 +14,10 @@ class RMSNorm(Norm):
     without the spec's ``weight_suffix`` (".weight")."""
 
     graph_safe = True
+    _ones = None
     takes_shares = True        # the kernel adds a product's unadded shares while it reads them
     takes_post = True          # ... and norms and scales the delta first where a layer asks for that
+    takes_streams = True       # ... and has a kernel that reads several streams as one vector
     takes_stream = True        # ... and can leave the normed row in the stream (a layer whose norm comes after the sum)
 
     def param_specs(self):
@@ -50,12 +52,26 @@ class RMSNorm(Norm):
         return out
 
 
+    def over_streams(self, stream, w_in, rows=None, store=True, conv=None, tail=None, ctx=None):
+        if self.spec.groups != 1:
+            raise ValueError("rmsnorm: groups are not built over several streams")
+        if w_in is None:
+            w_in = self._ones if self._ones is not None and self._ones.numel() == stream.x.shape[1] else None
+            if w_in is None:
+                w_in = self._ones = torch.ones(stream.x.shape[1], dtype=torch.float32, device=stream.x.device)
+        n = stream.x.shape[0] if rows is None else rows.numel()
+        out = torch.empty((n, self.spec.size), dtype=self.rt.dtype, device=stream.x.device)
+        return self.rt.ops.streams_norm(stream.x, w_in, self.weight, self.spec.eps, out, change=stream.take(), rows=rows, store=store,
+                                        conv=conv, tail=tail, ctx=ctx, status=stream.status)
+
+
 @register_part("norm", "layernorm")
 class LayerNorm(RMSNorm):
     """out = w * (v - mean(v)) * rsqrt(var(v) + eps) with v = x (+ delta), var the mean of the squared deviations, no
     bias; everything in 32-bit and one rounding at the end.  The kernel is the RMS norm's with the mean taken off."""
 
     takes_stream = False
+    takes_streams = False
 
     def __init__(self, spec, prefix, rt):
         super().__init__(spec, prefix, rt)

@@ -147,7 +147,9 @@ class LatentAttentionSpec(MixerSpec):
     ``rot_dim`` rotated].  D_kv h has ``kv_rank`` + ``rot_dim`` rows: the first, normed the same way, are the latent c; the
     others, rotated and not normed, are a key part that all heads share.  Head i's key is [U_k,i c | shared part], its value
     U_v,i c (``v_dim``); score = q . k * ``scale``; causal softmax, with ``sink`` one more term exp(s_i) (a number a head) in
-    the denominator; with ``gate`` the heads' results are multiplied by sigmoid(G h); then the output projection.
+    the denominator; ``gate`` "element": the heads' results are multiplied element by element by sigmoid(G h), "head": head
+    i's by sigmoid(G h)_i (G [heads, hidden]); then the output projection.  ``window`` None sees all earlier tokens; w sees
+    token j from position p if p - w < j <= p.
     ``names``: D_q, its norm, U_q, D_kv, its norm, U_k, U_v, output, sink, gate."""
     hidden: int = 0
     heads: int = 0
@@ -158,7 +160,8 @@ class LatentAttentionSpec(MixerSpec):
     kv_rank: int = 0
     scale: float = 1.0
     sink: bool = False
-    gate: bool = False
+    gate: str = "none"
+    window: Optional[int] = None
     norm_eps: float = 1e-6
     position: PositionSpec = field(default_factory=lambda: PositionSpec(kind="none"))
     names: Tuple[str, ...] = ("dq", "dq.norm", "uq", "dkv", "dkv.norm", "uk", "uv", "o", "sink", "g")
@@ -337,7 +340,12 @@ class ExpertsSpec(FeedForwardSpec):
     ``router``, ``e<i>.gate|up|down``, ``shared.gate|up|down`` below the part's prefix.
     ``activation`` "clamped": an expert's inner vector is g sigmoid(``gate_alpha`` g) (u + 1) with g = min(gate(x), ``limit``)
     and u = clamp(up(x), -``limit``, ``limit``) (the shared expert with ``shared_limit``).  ``router_weights`` "sigmoid_share":
-    the chosen experts weigh as sigmoid(z) over the chosen experts' sum of sigmoid(z) (+ 1e-20), times ``router_scale``."""
+    the chosen experts weigh as sigmoid(z) over the chosen experts' sum of sigmoid(z) (+ 1e-20), times ``router_scale``
+    ("softmax": the softmax over the chosen logits, which is the softmax over all logits divided by the chosen ones' sum of
+    it, times ``router_scale``).
+    ``activation`` "relu_square": the experts have no gate matrix, an expert is down(max(up(x), 0)^2).  ``shared_gate_name``: the
+    shared expert's result is multiplied by sigmoid(g . x), g [1, hidden] the tensor of that name below the part's prefix
+    (32-bit)."""
     hidden: int = 0
     experts: int = 0
     top: int = 1
@@ -353,6 +361,7 @@ class ExpertsSpec(FeedForwardSpec):
     router_name: str = "router"
     expert_prefix: str = "e"
     shared_prefix: str = "shared."
+    shared_gate_name: Optional[str] = None
     kind: str = "experts"
 
 
@@ -365,6 +374,12 @@ class BlockSpec:
     after the sums and their result is the stream.  With ``shift_name`` the mixer reads h_t + (h_(t-1) - h_t) * mu
     (mu [hidden] the tensor of that name below the layer's prefix, h_(t-1) the previous token's x, zeros before a request's
     first token), and the layer keeps a request's last x beside what its mixer keeps.
+
+    ``streams`` (the model's residual is several streams x_s): sublayer q = 1, 2 reads u = sum_s in[s] x_s and all streams
+    change at once, x_t <- sum_s mix[s, t] x_s + out[t] sublayer(h), h = norm(u); in, out [streams] and mix [streams, streams]
+    (from, to) are the tensors ``stream_prefixes[q - 1]`` + ``stream_names``.  With ``conv_taps`` n > 0 the sublayer reads
+    h + conv(h) instead, conv(h)_t = sum_j w[:, j] h_(t - n + 1 + j) with w [hidden, n] the tensor ``conv_names[q - 1]`` (zeros before
+    a request's first token); the layer keeps a request's last n - 1 rows h of either sublayer.
 
     ``prefix`` is the tensor-name prefix of the layer; ``mixer_prefix`` and the others
     are appended to it for the parts below it."""
@@ -385,6 +400,11 @@ class BlockSpec:
     residual_mult: float = 1.0
     stream_scale: float = 1.0
     shift_name: Optional[str] = None
+    streams: int = 0
+    stream_prefixes: Tuple[str, str] = ("hc1.", "hc2.")
+    stream_names: Tuple[str, str, str] = ("in", "out", "mix")
+    conv_taps: int = 0
+    conv_names: Tuple[str, str] = ("canon1", "canon2")
 
 
 @dataclass(frozen=True)
@@ -405,12 +425,21 @@ class RunSpec:
 
 @dataclass(frozen=True)
 class EmbeddingSpec:
-    """How token ids become the residual stream.  ``table``: x[t] = scale * table[id[t]] in 32-bit."""
+    """How token ids become the residual stream.  ``table``: x[t] = scale * table[id[t]] in 32-bit.
+    ``pair``: x[t] = N(table[id[t]] + second[row[t]]) with ``pair`` = (buckets, a, b), row[t] = (id[t - 1] a + id[t] b) mod buckets, and
+    row number ``buckets`` for a request's first token; second [buckets + 1, hidden] the tensor ``pair_name``, N the norm
+    ``norm`` (weight ``norm_name``; None: nothing).  ``streams``: how many streams the residual has (0: it is no bundle of
+    streams); each takes the result."""
     vocab: int
     hidden: int
     name: str = "model.embed_tokens.weight"
     scale: float = 1.0
     kind: str = "table"
+    pair: Optional[Tuple[int, int, int]] = None
+    pair_name: str = "pairs"
+    norm: Optional[NormSpec] = None
+    norm_name: str = "model.embed_norm"
+    streams: int = 0
 
 
 @dataclass(frozen=True)
@@ -440,6 +469,10 @@ class ModelSpec:
     embedding: EmbeddingSpec
     head: HeadSpec
     max_positions: int = 0
+    # the residual is a bundle of that many streams (0: one stream, no bundle); every block is then of the kind "streams"
+    streams: int = 0
+    # the cache slot of what the embedding keeps of a request (None: it keeps nothing)
+    embedding_cache: Optional[int] = None
     # patterns (fnmatch) of tensor names that a checkpoint of the architecture may hold and the model does not read
     ignored: Tuple[str, ...] = ()
     # token ids at which generation ends unless a request says otherwise (from the architecture's configuration)
