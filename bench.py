@@ -445,6 +445,22 @@ def _fosepel_config(width, ff, mem, att, delta):
     return {"architecture": "Fosepel", "vocab": 32768, "width": width, "layers": layers, "norm": {"eps": 1e-6}, "logit_softcap": 30.0}
 
 
+def _laposun_config(width, ff, att, window, layers=4):
+    """``layers`` latent-attention layers under a window with a gate a head, four streams and convolutions of 4 taps; every
+    other layer has a dense feed-forward of ``ff``, the others 8 experts (square of relu) of which a token uses 2 beside a
+    gated shared expert, the three experts a token runs having 1.5 ``ff`` inner values together (as many weights as the
+    dense gated one).  ``att``: (heads, kv heads, head size) of the Qwen2 model of equal size; the latents as for Geponex."""
+    heads, dim = att[0], att[2]
+    inner = ff // 2 // 64 * 64
+    moe = {"kind": "moe", "router": {"experts": 8, "top": 2, "scale": 1.5}, "expert": {"ff": inner}, "shared": {"ff": inner}}
+    mixer = {"heads": heads, "dim": dim, "rot_dim": dim // 2, "vdim": dim, "q_rank": 12 * dim, "kv_rank": 4 * dim,
+             "scale": (1.5 * dim) ** -0.5, "rot": {"dims": dim // 2, "base": 1e6}, "mask": {"size": window}}
+    return {"architecture": "Laposun", "vocab": 32768, "width": width, "streams": 4, "canon": {"taps": 4}, "norm": {"eps": 1e-6},
+            "embedding": {"bigram": {"buckets": 20011, "mul_prev": 31, "mul_cur": 1009}},
+            "layers": [{"type": "latent_attention", "mixer": mixer, "mlp": {"kind": "dense", "ff": ff} if i % 2 == 0 else moe}
+                       for i in range(layers)]}
+
+
 DESIGN_SIZES = {
     # name: width, feed-forward, (gla heads, dim, vdim), (attention heads, kv heads, head size), (delta heads, dim), chunk
     "w1024": (1024, 4096, (8, 64, 128), (16, 2, 64), (8, 64), 1024),
@@ -458,7 +474,11 @@ DESIGNS = {
     "geponex": lambda width, ff, gla, att, delta, chunk: _geponex_config(width, ff, gla, att),
     # (the matrix memory has the gated linear attention's sizes)
     "fosepel": lambda width, ff, gla, att, delta, chunk: _fosepel_config(width, ff, gla, att, delta),
+    # (the window is the other design's chunk)
+    "laposun": lambda width, ff, gla, att, delta, chunk: _laposun_config(width, ff, att, chunk),
 }
+# a design whose mixers and experts are another design's with other options is measured beside that one too
+CLOSEST = {"laposun": "geponex"}
 
 
 def design_points(design: str, sizes, steps: int, warmup: int) -> int:
@@ -494,7 +514,7 @@ def design_points(design: str, sizes, steps: int, warmup: int) -> int:
     def per_kernel(runner, entries):
         """Device time of each of the package's kernels in one eager step, by the name of the op."""
         names = [n for n in ("embedding", "rmsnorm", "layernorm", "polynorm", "head_norm_gate", "gla_scan", "delta_scan",
-                             "retention_scan", "gated_delta_scan", "conv_tail_update", "memory_scan", "normed_sum", "add_rows", "route_experts", "route_topk", "token_shift", "latent_prepare", "head_matmul", "attention_latent", "xielu",
+                             "retention_scan", "gated_delta_scan", "conv_tail_update", "memory_scan", "embedding_pair", "streams_norm", "relu_square", "linear_relu_square", "expert_lists", "gather_picks", "combine_picks", "normed_sum", "add_rows", "route_experts", "route_topk", "token_shift", "latent_prepare", "head_matmul", "attention_latent", "xielu",
                              "gate_clamp", "attention_differential", "attention_prepare", "attention_general", "rope_store", "paged_attention", "rope_attention", "linear",
                              "linear_silu_mul", "linear_to_stream", "logits_scale_cap") if hasattr(ops, n)]
         saved, events = {n: getattr(ops, n) for n in names}, []
@@ -535,6 +555,8 @@ def design_points(design: str, sizes, steps: int, warmup: int) -> int:
                           num_hidden_layers=4, num_attention_heads=att[0], num_key_value_heads=att[1], head_dim=att[2],
                           rms_norm_eps=1e-6, rope_theta=1e6, max_position_embeddings=8192, tie_word_embeddings=True),
         }
+        if design in CLOSEST:
+            models[CLOSEST[design]] = DESIGNS[CLOSEST[design]](width, ff, gla, att, delta, chunk)
         res = {}
         for name, raw in models.items():
             cfg = config_from_dict(raw)
@@ -586,7 +608,7 @@ def design_points(design: str, sizes, steps: int, warmup: int) -> int:
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--design", default=None, help="instead of the default workload: prefill and decode throughput of this design "
-                    "('sisetar', 'vegilix', 'geponex', 'fosepel') at layer sizes that resemble a served model's, beside a Qwen2 model of equal size")
+                    "('sisetar', 'vegilix', 'geponex', 'fosepel', 'laposun') at layer sizes that resemble a served model's, beside a Qwen2 model of equal size")
     ap.add_argument("--design-sizes", default="w1024,w4096", help="which of the sizes of --design to run, with commas between them")
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=200)
