@@ -18,7 +18,9 @@ namespace vtb {
 
 namespace {
 constexpr int kMaxExperts = 1024;
-constexpr int kRouteThreads = 128;
+constexpr int kRouteThreads = 128;          // many tokens
+constexpr int kRouteFewThreads = 512;       // few tokens (a block's rows are long, and there are few blocks)
+constexpr int kRouteFewTokens = 296;
 }
 
 // The `top` largest of z[0 .. experts) (the lower index among equals), by the first warp of the block: picked[k] and
@@ -101,8 +103,9 @@ __device__ __forceinline__ void router_logits(float* z, const float* __restrict_
     }
 }
 
+// (Every block of a token, blockIdx.y, forms the token's weights and scales its share of the columns.)
 template <typename T>
-__global__ void __launch_bounds__(kRouteThreads)
+__global__ void __launch_bounds__(kRouteFewThreads)
 route_experts_kernel(const float* __restrict__ logits, const T* __restrict__ x, const float* __restrict__ router, int width,
                      int experts, int top, T* __restrict__ act, int act_stride, int inter, int mode, float scale,
                      const float* __restrict__ shared_gate) {
@@ -112,7 +115,7 @@ route_experts_kernel(const float* __restrict__ logits, const T* __restrict__ x, 
     __shared__ int picked[kMaxExperts];
     pdl_launch();
     pdl_wait();
-    const int t = blockIdx.x;
+    const int t = blockIdx.x, first = blockIdx.y * blockDim.x + threadIdx.x, stride = gridDim.y * blockDim.x;
     for (int e = threadIdx.x; e < experts; e += blockDim.x) w[e] = 0.f;
     router_logits(z, logits, x, router, width, experts, t, shared_gate);
     __syncthreads();
@@ -121,11 +124,11 @@ route_experts_kernel(const float* __restrict__ logits, const T* __restrict__ x, 
     T* row = act + (size_t)t * act_stride;
     if (shared_gate != nullptr) {
         const float g = 1.f / (1.f + expf(-z[experts]));
-        for (int c = experts * inter + threadIdx.x; c < act_stride; c += blockDim.x) row[c] = from_float<T>(to_float(row[c]) * g);
+        for (int c = experts * inter + first; c < act_stride; c += stride) row[c] = from_float<T>(to_float(row[c]) * g);
     }
     if (inter % 8 == 0 && act_stride % 8 == 0 && (reinterpret_cast<uintptr_t>(act) & 15) == 0) {
         const int per = inter / 8;
-        for (int c = threadIdx.x; c < experts * per; c += blockDim.x) {
+        for (int c = first; c < experts * per; c += stride) {
             const float we = w[c / per];
             float v[8];
             if (we != 0.f) {
@@ -140,7 +143,7 @@ route_experts_kernel(const float* __restrict__ logits, const T* __restrict__ x, 
         }
         return;
     }
-    for (int c = threadIdx.x; c < experts * inter; c += blockDim.x) {
+    for (int c = first; c < experts * inter; c += stride) {
         const float we = w[c / inter];
         row[c] = from_float<T>(we != 0.f ? to_float(row[c]) * we : 0.f);
     }
@@ -300,10 +303,13 @@ cudaError_t launch_route_experts(int dtype, const float* logits, const void* x, 
     if (n_tokens == 0) return cudaSuccess;
     if (shared_gate != nullptr && x == nullptr) return cudaErrorInvalidValue;
     if (experts < 1 || experts > kMaxExperts || top < 1 || top > experts || (x != nullptr && width % 8)) return cudaErrorInvalidValue;
+    const bool few = n_tokens <= kRouteFewTokens;
+    const int threads = few ? kRouteFewThreads : kRouteThreads;
+    const dim3 grid(n_tokens, few ? max(1, min(min(4, 296 / n_tokens), act_stride / (8 * threads))) : 1);
     if (dtype == kBF16)
-        return launch(route_experts_kernel<__nv_bfloat16>, n_tokens, kRouteThreads, 0, stream, logits, (const __nv_bfloat16*)x, router, width,
+        return launch(route_experts_kernel<__nv_bfloat16>, grid, threads, 0, stream, logits, (const __nv_bfloat16*)x, router, width,
                       experts, top, (__nv_bfloat16*)act, act_stride, inter, mode, scale, shared_gate);
-    return launch(route_experts_kernel<float>, n_tokens, kRouteThreads, 0, stream, logits, (const float*)x, router, width, experts, top,
+    return launch(route_experts_kernel<float>, grid, threads, 0, stream, logits, (const float*)x, router, width, experts, top,
                   (float*)act, act_stride, inter, mode, scale, shared_gate);
 }
 

@@ -82,14 +82,16 @@ __device__ __forceinline__ void turn_pair(float u, float v, int pos, float f, fl
 // written to cq [tokens, cq_stride] (columns beyond q_rank are left).  The first kv_rank numbers at kv_col are normed
 // the same way with k_weight, the last rot_dim are rotated by the token's position (the first 2 * half of them; not
 // normed), and both go into the token's row of the page [pages, 1, page_size, kv_rank + rot_dim] if `store`.
-template <typename T>
+// VEC: eight values a thread at a time (every column, size and stride a multiple of 8).  Both sums of squares are formed
+// in one pass; their order depends on the sizes only.
+template <typename T, bool VEC>
 __global__ void latent_prepare_kernel(const T* __restrict__ y, int stride, int q_col, int q_rank, int kv_col, int kv_rank, int rot_dim,
                                       const float* __restrict__ q_weight, const float* __restrict__ k_weight, float eps,
                                       const float* __restrict__ freq, int half, float mult, const int* __restrict__ positions,
                                       const int* __restrict__ token_seq, const int* __restrict__ block_table, int table_stride,
                                       int n_seqs, int n_pages, int page_size, T* __restrict__ cq, int cq_stride, T* __restrict__ pages,
                                       int store, int* status) {
-    __shared__ float scratch[32];
+    __shared__ float scratch[2][32];
     pdl_launch();
     const int t = blockIdx.x;
     const int seq = token_seq[t];
@@ -111,25 +113,49 @@ __global__ void latent_prepare_kernel(const T* __restrict__ y, int stride, int q
         store = 0;
     }
     const T* row = y + (size_t)t * stride;
-    // the queries' latent
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < q_rank; i += blockDim.x) {
-        const float v = to_float(row[q_col + i]);
-        ss = fmaf(v, v, ss);
+    constexpr int N = VEC ? 8 : 1;
+    auto squares = [&](const T* p, int n) {
+        float ss = 0.f;
+        for (int i = threadIdx.x * N; i < n; i += blockDim.x * N) {
+            float v[8];
+            if constexpr (VEC) Vec8<T>::load(p + i, v);
+            else v[0] = to_float(p[i]);
+#pragma unroll
+            for (int j = 0; j < N; ++j) ss = fmaf(v[j], v[j], ss);
+        }
+        return ss;
+    };
+    auto scaled = [&](const T* p, int n, float r, const float* w, T* o) {
+        for (int i = threadIdx.x * N; i < n; i += blockDim.x * N) {
+            float v[8], u[8];
+            if constexpr (VEC) {
+                Vec8<T>::load(p + i, v);
+                Vec8<float>::load(w + i, u);
+            } else {
+                v[0] = to_float(p[i]);
+                u[0] = w[i];
+            }
+#pragma unroll
+            for (int j = 0; j < N; ++j) v[j] = v[j] * r * u[j];
+            if constexpr (VEC) Vec8<T>::store(o + i, v);
+            else o[i] = from_float<T>(v[0]);
+        }
+    };
+    // the queries' latent, and the keys' and values'
+    const float sq = warp_sum(squares(row + q_col, q_rank)), sk = warp_sum(store ? squares(row + kv_col, kv_rank) : 0.f);
+    const int lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
+    if (lane == 0) {
+        scratch[0][threadIdx.x >> 5] = sq;
+        scratch[1][threadIdx.x >> 5] = sk;
     }
-    const float rq = rsqrtf(block_sum(ss, scratch) / (float)q_rank + eps);
-    for (int i = threadIdx.x; i < q_rank; i += blockDim.x)
-        cq[(size_t)t * cq_stride + i] = from_float<T>(to_float(row[q_col + i]) * rq * q_weight[i]);
+    __syncthreads();
+    const float rq = rsqrtf(warp_sum(lane < n_warps ? scratch[0][lane] : 0.f) / (float)q_rank + eps);
+    const float rk = rsqrtf(warp_sum(lane < n_warps ? scratch[1][lane] : 0.f) / (float)kv_rank + eps);
+    scaled(row + q_col, q_rank, rq, q_weight, cq + (size_t)t * cq_stride);
     if (!store) return;
-    // the keys' and values' latent, and the shared rotated key part
-    ss = 0.f;
-    for (int i = threadIdx.x; i < kv_rank; i += blockDim.x) {
-        const float v = to_float(row[kv_col + i]);
-        ss = fmaf(v, v, ss);
-    }
-    const float rk = rsqrtf(block_sum(ss, scratch) / (float)kv_rank + eps);
     T* dst = pages + ((size_t)page * page_size + pos % page_size) * (kv_rank + rot_dim);
-    for (int i = threadIdx.x; i < kv_rank; i += blockDim.x) dst[i] = from_float<T>(to_float(row[kv_col + i]) * rk * k_weight[i]);
+    scaled(row + kv_col, kv_rank, rk, k_weight, dst);
+    // the shared rotated key part
     const T* kr = row + kv_col + kv_rank;
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
         float a, b;
@@ -147,15 +173,39 @@ cudaError_t launch_latent_prepare(int dtype, const void* y, int stride, int q_co
                                   cudaStream_t stream) {
     if (n_tokens == 0) return cudaSuccess;
     if (2 * half > rot_dim) return cudaErrorInvalidValue;
-    const int widest = max(q_rank, kv_rank);
-    const int threads = min(512, max(32, ((widest + 31) / 32) * 32));
+    const bool vec = stride % 8 == 0 && q_col % 8 == 0 && q_rank % 8 == 0 && kv_col % 8 == 0 && kv_rank % 8 == 0 && rot_dim % 8 == 0 &&
+                     cq_stride % 8 == 0 && ((uintptr_t)y & 15) == 0 && ((uintptr_t)cq & 15) == 0 && ((uintptr_t)pages & 15) == 0 &&
+                     ((uintptr_t)q_weight & 15) == 0 && ((uintptr_t)k_weight & 15) == 0;
+    const int widest = max(max(q_rank, kv_rank) / (vec ? 8 : 1), 2 * half);
+    const int threads = min(vec ? 256 : 512, max(32, ((widest + 31) / 32) * 32));
     if (dtype == kBF16)
-        return launch(latent_prepare_kernel<__nv_bfloat16>, n_tokens, threads, 0, stream, (const __nv_bfloat16*)y, stride, q_col, q_rank,
-                      kv_col, kv_rank, rot_dim, q_weight, k_weight, eps, freq, half, mult, positions, token_seq, block_table, table_stride,
-                      n_seqs, n_pages, page_size, (__nv_bfloat16*)cq, cq_stride, (__nv_bfloat16*)pages, store, status);
-    return launch(latent_prepare_kernel<float>, n_tokens, threads, 0, stream, (const float*)y, stride, q_col, q_rank, kv_col, kv_rank,
-                  rot_dim, q_weight, k_weight, eps, freq, half, mult, positions, token_seq, block_table, table_stride, n_seqs, n_pages,
-                  page_size, (float*)cq, cq_stride, (float*)pages, store, status);
+        return launch(vec ? latent_prepare_kernel<__nv_bfloat16, true> : latent_prepare_kernel<__nv_bfloat16, false>, n_tokens, threads, 0,
+                      stream, (const __nv_bfloat16*)y, stride, q_col, q_rank, kv_col, kv_rank, rot_dim, q_weight, k_weight, eps, freq, half,
+                      mult, positions, token_seq, block_table, table_stride, n_seqs, n_pages, page_size, (__nv_bfloat16*)cq, cq_stride,
+                      (__nv_bfloat16*)pages, store, status);
+    return launch(vec ? latent_prepare_kernel<float, true> : latent_prepare_kernel<float, false>, n_tokens, threads, 0, stream, (const float*)y,
+                  stride, q_col, q_rank, kv_col, kv_rank, rot_dim, q_weight, k_weight, eps, freq, half, mult, positions, token_seq, block_table,
+                  table_stride, n_seqs, n_pages, page_size, (float*)cq, cq_stride, (float*)pages, store, status);
+}
+
+// The rotated part of a head's inputs (`tail` numbers behind its `inner` ones) for n tokens from t0 on: pairs (2i, 2i + 1), the
+// first `half` of them turned by the token's position, copied behind the head's `outer` outputs.  Shared by `shares` CTAs,
+// of which this is number `share`.
+template <typename T>
+__device__ __forceinline__ void turn_tail(const T* __restrict__ x, size_t x_stride, T* __restrict__ out, size_t out_stride, int t0, int n, int tail,
+                                          const float* __restrict__ freq, int half, float mult, const int* __restrict__ positions,
+                                          const int* __restrict__ token_seq, int share, int shares) {
+    const int pairs = (tail + 1) / 2;
+    for (int e = share * blockDim.x + threadIdx.x; e < n * pairs; e += shares * blockDim.x) {
+        const int t = t0 + e / pairs, pair = e % pairs, i = 2 * pair;
+        const T* src = x + (size_t)t * x_stride + i;
+        T* dst = out + (size_t)t * out_stride + i;
+        const float u = to_float(src[0]), v = i + 1 < tail ? to_float(src[1]) : 0.f;
+        float a = u, b = v;
+        if (pair < half && token_seq[t] >= 0) turn_pair(u, v, positions[t], freq[pair], mult, a, b);
+        dst[0] = from_float<T>(a);
+        if (i + 1 < tail) dst[1] = from_float<T>(b);
+    }
 }
 
 // ------------------------------------------------------------------------- a product of each head with its own matrix
@@ -213,20 +263,9 @@ head_matmul_kernel(const T* __restrict__ x, int x_stride, int x_col, int x_head,
             out[(size_t)(t0 + tk) * out_stride + out_col + h * out_head + j] = from_float<T>(v);
         }
     }
-    if (mode != 1 || blockIdx.z != 0) return;
-    // the head's rotated part, behind its outputs
-    for (int e = threadIdx.x; e < n * tail; e += kHeadCols) {
-        const int tk = e / tail, i = e % tail, t = t0 + tk;
-        const T* src = x + (size_t)t * x_stride + x_col + h * x_head + inner;
-        float v = to_float(src[i]);
-        if (i < 2 * half && token_seq[t] >= 0) {
-            float a, b;
-            const int pair = i >> 1;
-            turn_pair(to_float(src[2 * pair]), to_float(src[2 * pair + 1]), positions[t], freq[pair], mult, a, b);
-            v = (i & 1) ? b : a;
-        }
-        out[(size_t)t * out_stride + out_col + h * out_head + outer + i] = from_float<T>(v);
-    }
+    if (mode == 1)
+        turn_tail(x + x_col + (size_t)h * x_head + inner, x_stride, out + out_col + (size_t)h * out_head + outer, out_stride, t0, n, tail, freq, half,
+                  mult, positions, token_seq, blockIdx.z, gridDim.z);
 }
 
 // The same product on the tensor cores (bfloat16, 32-bit sums, one rounding), for steps with many tokens: a CTA forms 64
@@ -310,23 +349,114 @@ head_matmul_mma_kernel(const __nv_bfloat16* __restrict__ x, int x_stride, int x_
             *reinterpret_cast<uint32_t*>(op + j) = pack_bf16(v0, v1);
         }
     }
-    if (mode != 1 || blockIdx.z != 0) return;
-    // the head's rotated part, behind its outputs
-    for (int e = threadIdx.x; e < n * tail; e += 128) {
-        const int tk = e / tail, i = e % tail, t = t0 + tk;
-        const __nv_bfloat16* src = x + (size_t)t * x_stride + x_col + h * x_head + inner;
-        float v = __bfloat162float(src[i]);
-        if (i < 2 * half && token_seq[t] >= 0) {
-            float a, b;
-            const int pair = i >> 1;
-            turn_pair(__bfloat162float(src[2 * pair]), __bfloat162float(src[2 * pair + 1]), positions[t], freq[pair], mult, a, b);
-            v = (i & 1) ? b : a;
-        }
-        out[(size_t)t * out_stride + out_col + h * out_head + outer + i] = __float2bfloat16_rn(v);
-    }
+    if (mode == 1)
+        turn_tail(x + x_col + (size_t)h * x_head + inner, x_stride, out + out_col + (size_t)h * out_head + outer, out_stride, t0, n, tail, freq, half,
+                  mult, positions, token_seq, blockIdx.z, gridDim.z);
 }
 
-// from how many tokens on a step's products of the heads run on the tensor cores (below, M_h's bytes bound the time)
+// The same product for steps with few tokens (up to 64), where the time is the latency of fetching M_h: a CTA forms all tokens x
+// 32 outputs of one head, so that a head's matrix comes through many CTAs at once, whole, in one wave of cp.async copies;
+// its four warps take every fourth step of 16 inner numbers and meet in shared memory, where their sums are added in the
+// order of the warps.  MT: tiles of 16 tokens.
+constexpr int kHfCols = 32;
+
+template <int MT>
+__global__ void __launch_bounds__(128)
+head_matmul_few_kernel(const __nv_bfloat16* __restrict__ x, int x_stride, int x_col, int x_head, const __nv_bfloat16* __restrict__ m,
+                       int inner, int outer, __nv_bfloat16* __restrict__ out, int out_stride, int out_col, int out_head, int n_tokens,
+                       int mode, int tail, const float* __restrict__ freq, int half, float mult, const int* __restrict__ positions,
+                       const int* __restrict__ token_seq, const __nv_bfloat16* __restrict__ gate, int gate_stride, int gate_col) {
+    constexpr int ROWS = 16 * MT, LB = kHfCols + 8, LS = kHfCols + 1;
+    const int steps = (inner + 15) / 16, LA = steps * 16 + 8;
+    extern __shared__ __align__(16) unsigned char hf_smem[];
+    __nv_bfloat16* bs = reinterpret_cast<__nv_bfloat16*>(hf_smem);           // [steps * 16][LB]
+    __nv_bfloat16* as = bs + (size_t)steps * 16 * LB;                        // [ROWS][LA]
+    float* sums = reinterpret_cast<float*>(as + (size_t)ROWS * LA);          // [4 warps][ROWS][LS]
+    pdl_launch();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gq = lane >> 2, tq = lane & 3;
+    const int h = blockIdx.x, n0 = blockIdx.y * kHfCols;
+    // the matrix is a weight, written by no kernel of the step: its copies start before the wait
+    const __nv_bfloat16* mh = m + (size_t)h * inner * outer + n0;
+    for (int c = threadIdx.x; c < steps * 16 * (kHfCols / 8); c += 128) {
+        const int r = c / (kHfCols / 8), piece = c % (kHfCols / 8);
+        const bool ok = r < inner && n0 + piece * 8 < outer;
+        cp_async16(bs + (size_t)r * LB + piece * 8, mh + (ok ? (size_t)r * outer + piece * 8 : 0), ok);
+    }
+    cp_async_commit();
+    pdl_wait();
+    const __nv_bfloat16* xh = x + x_col + (size_t)h * x_head;
+    const int pieces = steps * 2;
+    for (int c = threadIdx.x; c < ROWS * pieces; c += 128) {
+        const int r = c / pieces, piece = c % pieces;
+        const bool ok = r < n_tokens && piece * 8 < inner;
+        cp_async16(as + (size_t)r * LA + piece * 8, xh + (ok ? (size_t)r * x_stride + piece * 8 : 0), ok);
+    }
+    cp_async_commit();
+    cp_async_wait<0>();
+    __syncthreads();
+    float acc[MT][kHfCols / 8][4];
+#pragma unroll
+    for (int i = 0; i < MT; ++i)
+#pragma unroll
+        for (int j = 0; j < kHfCols / 8; ++j) acc[i][j][0] = acc[i][j][1] = acc[i][j][2] = acc[i][j][3] = 0.f;
+    const int mat = lane >> 3, r8 = lane & 7;
+    for (int kk = warp; kk < steps; kk += 4) {
+        uint32_t bf[kHfCols / 16][4];
+#pragma unroll
+        for (int dn = 0; dn < kHfCols / 16; ++dn)
+            ldmatrix_x4_trans(bf[dn], bs + (size_t)(kk * 16 + (mat & 1) * 8 + r8) * LB + dn * 16 + (mat >> 1) * 8);
+#pragma unroll
+        for (int i = 0; i < MT; ++i) {
+            uint32_t af[4];
+            ldmatrix_x4(af, as + (size_t)(i * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LA + kk * 16 + (lane >> 4) * 8);
+#pragma unroll
+            for (int dn = 0; dn < kHfCols / 16; ++dn) {
+                mma_bf16(acc[i][2 * dn], af, bf[dn][0], bf[dn][1]);
+                mma_bf16(acc[i][2 * dn + 1], af, bf[dn][2], bf[dn][3]);
+            }
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < MT; ++i)
+#pragma unroll
+        for (int nt = 0; nt < kHfCols / 8; ++nt)
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+                sums[((size_t)warp * ROWS + i * 16 + gq + 8 * (e >> 1)) * LS + nt * 8 + 2 * tq + (e & 1)] = acc[i][nt][e];
+    __syncthreads();
+    for (int e = threadIdx.x; e < n_tokens * kHfCols; e += 128) {
+        const int tk = e / kHfCols, c = e % kHfCols, j = n0 + c;
+        if (j >= outer) continue;
+        float v = 0.f;
+#pragma unroll
+        for (int w = 0; w < 4; ++w) v += sums[((size_t)w * ROWS + tk) * LS + c];
+        if (mode >= 2 && gate != nullptr)
+            v *= 1.f / (1.f + expf(-__bfloat162float(gate[(size_t)tk * gate_stride + gate_col + (mode == 3 ? h : h * outer + j)])));
+        out[(size_t)tk * out_stride + out_col + (size_t)h * out_head + j] = __float2bfloat16_rn(v);
+    }
+    if (mode == 1)
+        turn_tail(x + x_col + (size_t)h * x_head + inner, x_stride, out + out_col + (size_t)h * out_head + outer, out_stride, 0, n_tokens, tail, freq,
+                  half, mult, positions, token_seq, blockIdx.y, gridDim.y);
+}
+
+constexpr int kHfMaxTokens = 64;
+constexpr int kHfMaxBytes = 200 * 1024;
+
+static int head_matmul_few_bytes(int inner, int tiles) {
+    const int steps = (inner + 15) / 16;
+    return steps * 16 * (kHfCols + 8) * 2 + 16 * tiles * (steps * 16 + 8) * 2 + 4 * 16 * tiles * (kHfCols + 1) * 4;
+}
+
+template <int MT, typename... Args>
+static cudaError_t launch_head_matmul_few(dim3 grid, int bytes, cudaStream_t stream, Args... args) {
+    static std::atomic<unsigned long long> done{0};
+    const cudaError_t e = allow_dynamic_smem(head_matmul_few_kernel<MT>, kHfMaxBytes, done);
+    if (e != cudaSuccess) return e;
+    return launch(head_matmul_few_kernel<MT>, grid, dim3(128), bytes, stream, args...);
+}
+
+// from how many tokens on a step's products of the heads run on the tensor cores where the kernel for few tokens does not take
+// their sizes
 constexpr int kHmMinTokens = 32;
 
 cudaError_t launch_head_matmul(int dtype, int m_dtype, const void* x, int x_stride, int x_col, int x_head, const void* m, int heads,
@@ -336,9 +466,23 @@ cudaError_t launch_head_matmul(int dtype, int m_dtype, const void* x, int x_stri
     if (n_tokens == 0 || heads == 0) return cudaSuccess;
     if (2 * half > tail || (mode == 1 && half > 0 && (freq == nullptr || positions == nullptr || token_seq == nullptr)))
         return cudaErrorInvalidValue;
-    if (dtype == kBF16 && m_dtype == kBF16 && n_tokens >= kHmMinTokens && inner % 8 == 0 && outer % 8 == 0 && x_stride % 8 == 0 &&
-        x_col % 8 == 0 && x_head % 8 == 0 && out_stride % 2 == 0 && out_col % 2 == 0 && out_head % 2 == 0 &&
-        ((uintptr_t)x & 15) == 0 && ((uintptr_t)m & 15) == 0 && ((uintptr_t)out & 3) == 0) {
+    const bool aligned = dtype == kBF16 && m_dtype == kBF16 && inner % 8 == 0 && outer % 8 == 0 && x_stride % 8 == 0 && x_col % 8 == 0 &&
+                         x_head % 8 == 0 && out_stride % 2 == 0 && out_col % 2 == 0 && out_head % 2 == 0 && ((uintptr_t)x & 15) == 0 &&
+                         ((uintptr_t)m & 15) == 0 && ((uintptr_t)out & 3) == 0;
+    const int few_tiles = n_tokens <= 16 ? 1 : n_tokens <= 32 ? 2 : 4;
+    if (aligned && n_tokens <= kHfMaxTokens && head_matmul_few_bytes(inner, few_tiles) <= kHfMaxBytes) {
+        const dim3 grid_few(heads, (outer + kHfCols - 1) / kHfCols);
+        const int few_bytes = head_matmul_few_bytes(inner, few_tiles);
+        auto run = [&](auto launcher) {
+            return launcher(grid_few, few_bytes, stream, (const __nv_bfloat16*)x, x_stride, x_col, x_head, (const __nv_bfloat16*)m, inner, outer,
+                            (__nv_bfloat16*)out, out_stride, out_col, out_head, n_tokens, mode, tail, freq, half, mult, positions, token_seq,
+                            (const __nv_bfloat16*)gate, gate_stride, gate_col);
+        };
+        if (few_tiles == 1) return run([](auto... a) { return launch_head_matmul_few<1>(a...); });
+        if (few_tiles == 2) return run([](auto... a) { return launch_head_matmul_few<2>(a...); });
+        return run([](auto... a) { return launch_head_matmul_few<4>(a...); });
+    }
+    if (aligned && n_tokens >= kHmMinTokens) {
         const dim3 grid_mma((n_tokens + kHmRows - 1) / kHmRows, heads, (outer + kHmCols - 1) / kHmCols);
         return launch(head_matmul_mma_kernel, grid_mma, 128, 0, stream, (const __nv_bfloat16*)x, x_stride, x_col, x_head,
                       (const __nv_bfloat16*)m, inner, outer, (__nv_bfloat16*)out, out_stride, out_col, out_head, n_tokens, mode, tail, freq,

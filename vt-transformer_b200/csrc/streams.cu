@@ -169,6 +169,7 @@ template <typename T, int SC, bool CONV>
 __global__ void __launch_bounds__(kStreamThreads)
 streams_norm_kernel(const StreamsParams p, const T* __restrict__ delta, T* __restrict__ out) {
     constexpr int SM = SC > 0 ? SC : kMaxStreams;
+    constexpr int kNear = 3;             // rows before that are fetched ahead (more, with more taps, one after the other)
     __shared__ float scratch[32];
     __shared__ float mix_s[SM * SM], out_s[SM], in_s[SM];
     extern __shared__ __align__(16) float us[];           // [width] u, [width] the tail's part of the convolution
@@ -201,21 +202,34 @@ streams_norm_kernel(const StreamsParams p, const T* __restrict__ delta, T* __res
     const size_t stride = (size_t)p.n_tokens * width;
     float ss = 0.f;
     for (int i = threadIdx.x * 4; i < width; i += blockDim.x * 4) {
-        float v[SM][4], u[4] = {0.f, 0.f, 0.f, 0.f};
+        // everything that is read comes before anything is written, so that the loads are in flight together
+        float v[SM][4], u[4] = {0.f, 0.f, 0.f, 0.f}, d[4] = {0.f, 0.f, 0.f, 0.f}, before[kNear][4];
 #pragma unroll
         for (int s = 0; s < SM; ++s)
             if (s < S) Vec4<float>::load(xt + (size_t)s * width + i, v[s]);
+        if (CONV && tail != nullptr) {
+#pragma unroll
+            for (int k = 0; k < kNear; ++k)
+                if (k < p.taps - 1) Vec4<float>::load(tail + (size_t)k * width + i, before[k]);
+        }
         if (change) {
-            float d[4] = {0.f, 0.f, 0.f, 0.f};
             if (delta != nullptr) {
                 Vec4<T>::load(delta + (size_t)t * width + i, d);
             } else {
-#pragma unroll 4
-                for (int q = 0; q < p.n_parts; ++q) {
-                    float e[4];
-                    Vec4<float>::load(p.parts + (size_t)t * width + i + q * stride, e);
+                for (int q0 = 0; q0 < p.n_parts; q0 += 4) {
+                    float e[4][4];
 #pragma unroll
-                    for (int j = 0; j < 4; ++j) d[j] += e[j];
+                    for (int q = 0; q < 4; ++q) {
+                        if (q0 + q < p.n_parts) {
+                            Vec4<float>::load(p.parts + (size_t)t * width + i + (q0 + q) * stride, e[q]);
+                        } else {
+                            e[q][0] = e[q][1] = e[q][2] = e[q][3] = 0.f;
+                        }
+                    }
+#pragma unroll
+                    for (int q = 0; q < 4; ++q)
+#pragma unroll
+                        for (int j = 0; j < 4; ++j) d[j] += e[q][j];
                 }
             }
 #pragma unroll
@@ -254,14 +268,23 @@ streams_norm_kernel(const StreamsParams p, const T* __restrict__ delta, T* __res
             // what the rows before add, and the tail one row on (its last row follows below)
             float c[4] = {0.f, 0.f, 0.f, 0.f};
             if (tail != nullptr) {
-#pragma unroll 3
-                for (int k = 0; k < p.taps - 1; ++k) {
+#pragma unroll
+                for (int k = 0; k < kNear; ++k) {
+                    if (k < p.taps - 1) {
+                        float w[4];
+                        Vec4<float>::load(p.conv + (size_t)k * width + i, w);
+#pragma unroll
+                        for (int j = 0; j < 4; ++j) c[j] = fmaf(w[j], before[k][j], c[j]);
+                        if (k > 0) Vec4<float>::store(tail + (size_t)(k - 1) * width + i, before[k]);
+                    }
+                }
+                for (int k = kNear; k < p.taps - 1; ++k) {
                     float h[4], w[4];
                     Vec4<float>::load(tail + (size_t)k * width + i, h);
                     Vec4<float>::load(p.conv + (size_t)k * width + i, w);
 #pragma unroll
                     for (int j = 0; j < 4; ++j) c[j] = fmaf(w[j], h[j], c[j]);
-                    if (k > 0) Vec4<float>::store(tail + (size_t)(k - 1) * width + i, h);
+                    Vec4<float>::store(tail + (size_t)(k - 1) * width + i, h);
                 }
             }
             Vec4<float>::store(us + width + i, c);

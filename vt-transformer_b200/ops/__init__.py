@@ -450,8 +450,27 @@ def attention_differential(y, q_col: int, out, out_col: int, out_scale: float, k
                                          sub_eps=sub_eps)
 
 
-LATENT_TARGET_CTAS = 296     # CTAs that the latent attention of a step of single tokens aims at (two for each SM)
-LATENT_MAX_RUNS = 16         # the most runs of keys that a sequence is cut into for that (the merge kernel's limit)
+LATENT_MAX_RUNS = 16         # the most runs of keys that the latent attention of a step of single tokens cuts a sequence into
+LATENT_RUN_COST = 3          # what a run costs beside its keys, in blocks of 32 keys (its queries, its end, its share of the merge)
+
+
+def _latent_runs(ctas: int, span: int, v_dim: int, device) -> int:
+    """Into how many runs a sequence's keys are cut, a CTA each, in a step of single tokens with ``ctas`` CTAs at one run: the
+    number with which the rounds of CTAs take the least time.  An SM holds two CTAs, or one where values have more than 256
+    numbers; a typical sequence is taken to hold three quarters of ``span`` keys (the bound of a captured graph lies
+    between a sequence's length and twice that)."""
+    sms = _sm_counts.get(device)
+    if sms is None:
+        sms = _sm_counts[device] = torch.cuda.get_device_properties(device).multi_processor_count
+    slots, blocks = sms * (1 if v_dim > 256 else 2), max(1.0, span * 0.75 / 32)
+    best, at = None, 1
+    for runs in range(1, LATENT_MAX_RUNS + 1):
+        if runs > 1 and 2 * runs > blocks:             # a run has two blocks or more
+            break
+        cost = -(-ctas * runs // slots) * (blocks / runs + LATENT_RUN_COST)
+        if best is None or cost < best - 1e-9:
+            best, at = cost, runs
+    return at
 
 
 def attention_latent(q, q_col: int, out, out_col: int, pages, ctx, block_table, heads: int, key: int, v_dim: int, scale: float,
@@ -473,10 +492,8 @@ def attention_latent(q, q_col: int, out, out_col: int, pages, ctx, block_table, 
         part = None
         if singles:
             # few sequences leave most SMs without a CTA: every sequence's keys are cut into runs, a CTA each
-            ctas = ctx.n_seqs * -(-int(heads) // rows)
-            runs = min(LATENT_MAX_RUNS, max(1, LATENT_TARGET_CTAS // ctas))
-            if window:          # (no more runs than the window's keys fill with two blocks of 32 each)
-                runs = max(1, min(runs, -(-_key_span(ctx.max_kv_len, int(window), 0) // 64)))
+            runs = _latent_runs(ctx.n_seqs * -(-int(heads) // rows), _key_span(ctx.max_kv_len, int(window) if window else 0, 0), int(v_dim),
+                                q.device)
             if runs > 1:
                 part = torch.empty((runs, q.shape[0], int(heads), int(v_dim) + 2), dtype=torch.float32, device=q.device)
         be.attention_latent(q, int(q_col), out, int(out_col), pages, ctx.cu_q, ctx.q_start, block_table, tiles, int(heads), int(key),
