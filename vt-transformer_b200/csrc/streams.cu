@@ -166,7 +166,7 @@ struct StreamsParams {
 // tail moves on by one row.  SC: the number of streams where it is known when compiled (0: p.S).  The sum of squares has an
 // order that depends on the width alone.
 template <typename T, int SC, bool CONV>
-__global__ void __launch_bounds__(kStreamThreads)
+__global__ void __launch_bounds__(kStreamThreads, CONV || SC == 0 ? 1 : 2)
 streams_norm_kernel(const StreamsParams p, const T* __restrict__ delta, T* __restrict__ out) {
     constexpr int SM = SC > 0 ? SC : kMaxStreams;
     constexpr int kNear = 3;             // rows before that are fetched ahead (more, with more taps, one after the other)
