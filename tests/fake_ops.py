@@ -177,13 +177,19 @@ def polynorm(z, coefficients, eps, out, n_mean=0):
     out.copy_((a * n(zf) + b * n(zf * zf) + c * n(zf * zf * zf) + e).to(out.dtype))
 
 
-def head_norm_gate(o, y, gate_col, weight, weight_per_channel, eps, act, out, out_col, out_scale, heads, v_dim, token_seq=None):
+def head_norm_gate(o, y, gate_col, weight, weight_per_channel, eps, act, out, out_col, out_scale, heads, v_dim, token_seq=None,
+                   gate_first=False):
     T = o.shape[0]
     oh = o.view(T, heads, v_dim)
+    if gate_first:
+        z = y[:, gate_col:gate_col + heads * v_dim].float().view(T, heads, v_dim)
+        oh = oh * (z * torch.sigmoid(z) if act == 0 else torch.sigmoid(z))
     n = oh * torch.rsqrt((oh * oh).mean(dim=-1, keepdim=True) + eps)
     w = weight.view(heads, v_dim) if weight_per_channel else weight.view(1, v_dim)
     g = y[:, gate_col:gate_col + heads * v_dim].float().view(T, heads, v_dim)
     g = g * torch.sigmoid(g) if act == 0 else torch.sigmoid(g)
+    if gate_first:
+        g = torch.ones_like(g)
     out[:, out_col:out_col + heads * v_dim] = (out_scale * n * w * g).reshape(T, heads * v_dim).to(out.dtype)
     if token_seq is not None:
         out[token_seq < 0, out_col:out_col + heads * v_dim] = 0
@@ -400,9 +406,11 @@ def _pick_weights(z, mode, scale):
     return s / (s.sum() + 1e-20) * scale
 
 
-def route_experts(logits, top, act, inter, x=None, router=None, mode=0, scale=1.0, shared_gate=None):
+def route_experts(logits, top, act, inter, x=None, router=None, mode=0, scale=1.0, shared_gate=None, bias=None):
     if logits is None:
         logits = x.float() @ router.float().t()
+    if bias is not None:
+        logits = logits + bias
     T, n = logits.shape
     w = torch.zeros((T, n), dtype=torch.float32)
     chosen = torch.zeros((T, n), dtype=torch.bool)
@@ -416,11 +424,13 @@ def route_experts(logits, top, act, inter, x=None, router=None, mode=0, scale=1.
         act[:, n * inter:] = (act[:, n * inter:].float() * torch.sigmoid(x.float() @ shared_gate)[:, None]).to(act.dtype)
 
 
-def route_topk(logits, top, ids, weights, x=None, router=None, mode=0, scale=1.0, shared_gate=None, gates=None):
+def route_topk(logits, top, ids, weights, x=None, router=None, mode=0, scale=1.0, shared_gate=None, gates=None, bias=None):
     if shared_gate is not None:
         gates.copy_(torch.sigmoid(x.float() @ shared_gate))
     if logits is None:
         logits = x.float() @ router.float().t()
+    if bias is not None:
+        logits = logits + bias
     for t in range(logits.shape[0]):
         order = sorted(range(logits.shape[1]), key=lambda e: (-float(logits[t, e]), e))[:top]
         ids[t] = torch.tensor(order, dtype=torch.int32)
@@ -688,3 +698,43 @@ def conv_rows(h, w, tail, cu_q, seq_rows, tiles, per_tile, out, status=None):
 
 def relu_square(z, out):
     out.copy_((z.float().clamp(min=0.0) ** 2).to(out.dtype))
+
+
+# ---- the kernels of a layer whose results are normed before they join the stream, and of the state-space recurrence ----
+
+
+def add_normed(x, delta, weight, eps, mult, out, compute_dtype):
+    if delta is not None:
+        d = delta.sum(dim=0) if delta.dim() == 3 else delta.float()
+        x += _normed_first(d, weight, eps, mult)
+    if out is not None:
+        out.copy_(x.to(out.dtype))
+
+
+def causal_conv(y, col, w, bias, silu, tail, cu_q, rows, tiles, per_tile, out, status=None):
+    taps, channels = w.shape
+    assert per_tile >= max(1, taps - 1)
+    for row, a, b in _sequences(cu_q, rows):
+        x = y[a:b, col:col + channels].float()
+        if taps > 1:
+            x = torch.cat([tail[row], x], dim=0)
+            tail[row] = x[-(taps - 1):].clone()
+        z = sum(x[j:j + b - a] * w[j] for j in range(taps))
+        if bias is not None:
+            z = z + bias
+        out[a:b] = (z * torch.sigmoid(z) if silu else z).to(out.dtype)
+
+
+def state_space_scan(u, y, dt_col, a_log, dt_bias, d, state, cu_q, rows, seqs, o, heads, groups, dim, v_dim, status=None):
+    listed = _sequences(cu_q, rows) if seqs is None else [_sequences(cu_q, rows)[int(i)] for i in seqs]
+    inner = heads * v_dim
+    for row, a, b in listed:
+        x = u[a:b, :inner].float().view(b - a, heads, v_dim)
+        B = u[a:b, inner:inner + groups * dim].float().view(b - a, groups, dim).repeat_interleave(heads // groups, dim=1)
+        C = u[a:b, inner + groups * dim:].float().view(b - a, groups, dim).repeat_interleave(heads // groups, dim=1)
+        step = torch.nn.functional.softplus(y[a:b, dt_col:dt_col + heads].float() + dt_bias, threshold=100.0)
+        S = state[row].clone()
+        for t in range(b - a):
+            S = torch.exp(-torch.exp(a_log) * step[t])[:, None, None] * S + (step[t][:, None] * B[t])[:, :, None] * x[t][:, None, :]
+            o[a + t] = (torch.einsum("hnp,hn->hp", S, C[t]) + d[:, None] * x[t]).reshape(-1)
+        state[row] = S

@@ -1,5 +1,6 @@
 from .base import ConfigError, KeyReader, ModelConfig
 from .fosepel import FosepelConfig
+from .gedulorn import GedulornConfig
 from .geponex import GeponexConfig
 from .laposun import LaposunConfig
 from .qwen2 import Qwen2Config

@@ -161,7 +161,7 @@ void check_cols(const Tensor& y, int64_t col, int64_t n, const char* what) {
 
 void head_norm_gate(const Tensor& o, const Tensor& y, int64_t gate_col, const Tensor& weight, bool weight_per_channel, double eps,
                     int64_t act, Tensor& out, int64_t out_col, double out_scale, int64_t heads, int64_t v_dim,
-                    c10::optional<Tensor> token_seq) {
+                    c10::optional<Tensor> token_seq, bool gate_first) {
     check_f32(o, "o"); check_cuda(y, "y"); check_cuda(out, "out"); check_f32(weight, "weight");
     TORCH_CHECK(o.dim() == 2 && y.dim() == 2 && out.dim() == 2 && o.size(1) == heads * v_dim && y.size(0) == o.size(0) && out.size(0) == o.size(0),
                 "head_norm_gate: o [tokens, heads * v_dim], y and out with as many rows");
@@ -174,7 +174,109 @@ void head_norm_gate(const Tensor& o, const Tensor& y, int64_t gate_col, const Te
     c10::cuda::CUDAGuard guard(o.device());
     check_launch(vtb::launch_head_norm_gate(dtype_code(y, "y"), o.data_ptr<float>(), y.data_ptr(), y.size(1), gate_col, weight.data_ptr<float>(),
                                             weight_per_channel, (float)eps, act, out.data_ptr(), out.size(1), out_col, (float)out_scale, ts,
-                                            o.size(0), heads, v_dim, stream_of(o)), "head_norm_gate");
+                                            o.size(0), heads, v_dim, stream_of(o), gate_first ? 1 : 0), "head_norm_gate");
+}
+
+void add_normed(Tensor& x, c10::optional<Tensor> delta, c10::optional<Tensor> weight, double eps, double mult, c10::optional<Tensor> out,
+                int64_t compute_dtype) {
+    check_f32(x, "x");
+    TORCH_CHECK(x.dim() == 2 && x.size(1) % 8 == 0, "add_normed: x [tokens, hidden], hidden a multiple of 8");
+    TORCH_CHECK(delta.has_value() || out.has_value(), "add_normed: something to add or to copy");
+    int code = (int)compute_dtype;
+    const void* dp = nullptr;
+    const float* pp = nullptr;
+    int n_parts = 0;
+    if (delta.has_value() && delta->dim() == 3) {
+        check_f32(*delta, "delta");
+        TORCH_CHECK(delta->size(0) >= 1 && delta->size(1) == x.size(0) && delta->size(2) == x.size(1), "add_normed: shares of a delta are [shares, tokens, hidden]");
+        pp = delta->data_ptr<float>();
+        n_parts = delta->size(0);
+    } else if (delta.has_value()) {
+        check_cuda(*delta, "delta");
+        TORCH_CHECK(delta->sizes() == x.sizes() && dtype_code(*delta, "delta") == code, "add_normed: delta has the shape of x and the compute dtype");
+        dp = delta->data_ptr();
+    }
+    const float* wp = nullptr;
+    if (delta.has_value()) {
+        TORCH_CHECK(weight.has_value(), "add_normed: a delta comes with its norm's weight");
+        check_f32(*weight, "weight");
+        TORCH_CHECK(weight->numel() == x.size(1), "add_normed: weight [hidden]");
+        wp = weight->data_ptr<float>();
+    }
+    void* op = nullptr;
+    if (out.has_value()) {
+        check_cuda(*out, "out");
+        TORCH_CHECK(out->sizes() == x.sizes() && dtype_code(*out, "out") == code, "add_normed: out has the shape of x and the compute dtype");
+        op = out->data_ptr();
+    }
+    c10::cuda::CUDAGuard guard(x.device());
+    check_launch(vtb::launch_add_normed(code, x.data_ptr<float>(), dp, pp, n_parts, wp, (float)eps, (float)mult, op, x.size(0), x.size(1),
+                                        stream_of(x)), "add_normed");
+}
+
+// ---- state-space mixers (state_space.cu)
+
+void causal_conv(const Tensor& y, int64_t col, const Tensor& w, c10::optional<Tensor> bias, bool silu, c10::optional<Tensor> tail, const Tensor& cu_q,
+                 const Tensor& rows, c10::optional<Tensor> tiles, int64_t per_tile, Tensor& out, c10::optional<Tensor> status) {
+    check_cuda(y, "y"); check_f32(w, "w"); check_i32(cu_q, "cu_q"); check_i32(rows, "rows"); check_cuda(out, "out");
+    TORCH_CHECK(y.dim() == 2 && w.dim() == 2 && out.dim() == 2 && out.size(0) == y.size(0) && out.size(1) == w.size(1) &&
+                out.scalar_type() == y.scalar_type(), "causal_conv: y [tokens, .], w [taps, channels], out [tokens, channels] of y's dtype");
+    const int64_t taps = w.size(0), channels = w.size(1);
+    TORCH_CHECK(taps >= 1 && taps <= 16 && per_tile >= 1 && per_tile >= taps - 1, "causal_conv: 1 to 16 taps, tiles of at least taps - 1 tokens");
+    TORCH_CHECK(col >= 0 && col + channels <= y.size(1), "causal_conv: the channels lie outside y");
+    TORCH_CHECK(cu_q.numel() == rows.numel() + 1, "causal_conv: cu_q has one entry more than rows");
+    const float* bp = nullptr;
+    if (bias.has_value()) { check_f32(*bias, "bias"); TORCH_CHECK(bias->numel() == channels, "causal_conv: bias [channels]"); bp = bias->data_ptr<float>(); }
+    float* tp = nullptr;
+    int state_rows = 0;
+    if (taps > 1) {
+        TORCH_CHECK(tail.has_value(), "causal_conv: more than one tap needs the kept inputs");
+        check_f32(*tail, "tail");
+        TORCH_CHECK(tail->dim() == 3 && tail->size(1) == taps - 1 && tail->size(2) == channels, "causal_conv: tail [rows, taps - 1, channels]");
+        tp = tail->data_ptr<float>();
+        state_rows = tail->size(0);
+    }
+    const int* lp = nullptr;
+    int n_tiles = rows.numel();
+    if (tiles.has_value()) {
+        check_i32(*tiles, "tiles");
+        TORCH_CHECK(tiles->dim() == 2 && tiles->size(1) == 2, "causal_conv: tiles [n, 2]");
+        lp = tiles->data_ptr<int>();
+        n_tiles = tiles->size(0);
+    }
+    c10::cuda::CUDAGuard guard(y.device());
+    check_launch(vtb::launch_causal_conv(dtype_code(y, "y"), y.data_ptr(), y.size(1), col, channels, w.data_ptr<float>(), taps, bp, silu ? 1 : 0, tp,
+                                         state_rows, cu_q.data_ptr<int>(), rows.data_ptr<int>(), rows.numel(), lp, n_tiles, per_tile,
+                                         out.data_ptr(), status_ptr(status), stream_of(y)), "causal_conv");
+}
+
+// what the state-space kernels share: u, the raw step sizes in y, a number a head each, the state
+void check_space(const Tensor& u, const Tensor& y, int64_t dt_col, const Tensor& a_log, const Tensor& dt_bias, const Tensor& d, const Tensor& state,
+                 const Tensor& cu_q, const Tensor& rows, const Tensor& o, int64_t heads, int64_t groups, int64_t dim, int64_t v_dim, const char* who) {
+    check_cuda(u, "u"); check_cuda(y, "y"); check_f32(a_log, "a_log"); check_f32(dt_bias, "dt_bias"); check_f32(d, "d"); check_f32(state, "state");
+    check_i32(cu_q, "cu_q"); check_i32(rows, "rows"); check_f32(o, "o");
+    TORCH_CHECK(groups >= 1 && heads % groups == 0 && dim >= 1 && dim <= 512, who, ": heads a multiple of groups, state sizes up to 512");
+    TORCH_CHECK(u.dim() == 2 && y.dim() == 2 && u.size(0) == y.size(0) && u.scalar_type() == y.scalar_type() &&
+                u.size(1) == heads * v_dim + 2 * groups * dim, who, ": u [tokens, heads * v_dim + 2 groups * dim] of y's dtype");
+    TORCH_CHECK(dt_col >= 0 && dt_col + heads <= y.size(1), who, ": the step sizes lie outside y");
+    TORCH_CHECK(a_log.numel() == heads && dt_bias.numel() == heads && d.numel() == heads, who, ": a_log, dt_bias and d [heads]");
+    TORCH_CHECK(state.dim() == 4 && state.size(1) == heads && state.size(2) == dim && state.size(3) == v_dim, who, ": state [rows, heads, dim, v_dim]");
+    TORCH_CHECK(o.dim() == 2 && o.size(0) == y.size(0) && o.size(1) == heads * v_dim, who, ": o [tokens, heads * v_dim]");
+    TORCH_CHECK(cu_q.numel() == rows.numel() + 1, who, ": cu_q has one entry more than rows");
+}
+
+void state_space_scan(const Tensor& u, const Tensor& y, int64_t dt_col, const Tensor& a_log, const Tensor& dt_bias, const Tensor& d, Tensor& state,
+                      const Tensor& cu_q, const Tensor& rows, c10::optional<Tensor> seqs, Tensor& o, int64_t heads, int64_t groups, int64_t dim,
+                      int64_t v_dim, c10::optional<Tensor> status) {
+    check_space(u, y, dt_col, a_log, dt_bias, d, state, cu_q, rows, o, heads, groups, dim, v_dim, "state_space_scan");
+    const int* sp = nullptr;
+    int listed = 0;
+    if (seqs.has_value()) { check_i32(*seqs, "seqs"); sp = seqs->data_ptr<int>(); listed = seqs->numel(); }
+    c10::cuda::CUDAGuard guard(y.device());
+    check_launch(vtb::launch_state_space_scan(dtype_code(y, "y"), u.data_ptr(), u.size(1), y.data_ptr(), y.size(1), dt_col, a_log.data_ptr<float>(),
+                                              dt_bias.data_ptr<float>(), d.data_ptr<float>(), state.data_ptr<float>(), state.size(0),
+                                              cu_q.data_ptr<int>(), rows.data_ptr<int>(), rows.numel(), sp, listed, o.data_ptr<float>(), heads,
+                                              groups, dim, v_dim, status_ptr(status), stream_of(y)), "state_space_scan");
 }
 
 void scale_into(const Tensor& src, Tensor& dst, int64_t dst_col, double scale) {
@@ -604,6 +706,14 @@ struct RouterInput {
     int width = 0, tokens = 0, experts = 0, x_dtype = vtb::kF32;
 };
 
+// a number for every expert that is added to its logit
+const float* router_bias(const c10::optional<Tensor>& bias, int experts, const char* who) {
+    if (!bias.has_value()) return nullptr;
+    check_f32(*bias, "bias");
+    TORCH_CHECK(bias->numel() == experts, who, ": a bias for every expert");
+    return bias->data_ptr<float>();
+}
+
 RouterInput router_input(const c10::optional<Tensor>& logits, const c10::optional<Tensor>& x, const c10::optional<Tensor>& router, const char* who,
                          const c10::optional<Tensor>& shared_gate) {
     RouterInput r;
@@ -632,7 +742,7 @@ RouterInput router_input(const c10::optional<Tensor>& logits, const c10::optiona
 }
 
 void route_topk(c10::optional<Tensor> logits, int64_t top, Tensor& ids, Tensor& weights, c10::optional<Tensor> x, c10::optional<Tensor> router,
-                int64_t mode, double scale, c10::optional<Tensor> shared_gate, c10::optional<Tensor> gates) {
+                int64_t mode, double scale, c10::optional<Tensor> shared_gate, c10::optional<Tensor> gates, c10::optional<Tensor> bias) {
     check_i32(ids, "ids"); check_f32(weights, "weights");
     const RouterInput r = router_input(logits, x, router, "route_topk", shared_gate);
     float* gp = nullptr;
@@ -647,7 +757,8 @@ void route_topk(c10::optional<Tensor> logits, int64_t top, Tensor& ids, Tensor& 
     TORCH_CHECK(r.experts <= 1024 && top >= 1 && top <= r.experts, "route_topk: 1 <= top <= experts <= 1024");
     c10::cuda::CUDAGuard guard(ids.device());
     check_launch(vtb::launch_route_topk(r.x_dtype, r.logits, r.x, r.router, r.width, r.tokens, r.experts, top, ids.data_ptr<int>(),
-                                        weights.data_ptr<float>(), stream_of(ids), (int)mode, (float)scale, r.shared_gate, gp), "route_topk");
+                                        weights.data_ptr<float>(), stream_of(ids), (int)mode, (float)scale, r.shared_gate, gp,
+                                        router_bias(bias, r.experts, "route_topk")), "route_topk");
 }
 
 void expert_lists(const Tensor& ids, Tensor& lists, Tensor& counts) {
@@ -694,7 +805,7 @@ void combine_picks(const Tensor& y, const Tensor& where, const Tensor& weights, 
 }
 
 void route_experts(c10::optional<Tensor> logits, int64_t top, Tensor& act, int64_t inter, c10::optional<Tensor> x, c10::optional<Tensor> router,
-                   int64_t mode, double scale, c10::optional<Tensor> shared_gate) {
+                   int64_t mode, double scale, c10::optional<Tensor> shared_gate, c10::optional<Tensor> bias) {
     check_cuda(act, "act");
     const RouterInput r = router_input(logits, x, router, "route_experts", shared_gate);
     TORCH_CHECK(act.dim() == 2 && act.size(0) == r.tokens, "route_experts: act [tokens, .]");
@@ -703,7 +814,8 @@ void route_experts(c10::optional<Tensor> logits, int64_t top, Tensor& act, int64
     TORCH_CHECK(inter >= 0 && r.experts * inter <= act.size(1), "route_experts: experts * inter columns lie outside act");
     c10::cuda::CUDAGuard guard(act.device());
     check_launch(vtb::launch_route_experts(dtype_code(act, "act"), r.logits, r.x, r.router, r.width, r.tokens, r.experts, top, act.data_ptr(),
-                                           act.size(1), inter, stream_of(act), (int)mode, (float)scale, r.shared_gate), "route_experts");
+                                           act.size(1), inter, stream_of(act), (int)mode, (float)scale, r.shared_gate,
+                                           router_bias(bias, r.experts, "route_experts")), "route_experts");
 }
 
 
@@ -864,7 +976,8 @@ void latent_prepare(const Tensor& y, int64_t q_col, int64_t q_rank, int64_t kv_c
     check_i32(token_seq, "token_seq"); check_i32(block_table, "block_table"); check_cuda(cq, "cq"); check_cuda(pages, "pages");
     TORCH_CHECK(y.dim() == 2 && cq.dim() == 2 && cq.size(0) == y.size(0) && cq.size(1) >= q_rank && cq.scalar_type() == y.scalar_type() &&
                 pages.scalar_type() == y.scalar_type(), "latent_prepare: y and cq [tokens, .] and the pages of one dtype");
-    check_cols(y, q_col, q_rank, "latent_prepare (queries' latent)"); check_cols(y, kv_col, kv_rank + rot_dim, "latent_prepare (keys' latent)");
+    check_cols(y, q_col, q_rank, "latent_prepare (queries' latent)");
+    if (store) check_cols(y, kv_col, kv_rank + rot_dim, "latent_prepare (keys' latent)");      // else the columns are not read
     TORCH_CHECK(pages.dim() == 4 && pages.size(1) == 1 && pages.size(3) == kv_rank + rot_dim, "latent_prepare: pages [pages, 1, page_size, kv_rank + rot_dim]");
     TORCH_CHECK(q_weight.numel() == q_rank && k_weight.numel() == kv_rank, "latent_prepare: a weight for each latent");
     TORCH_CHECK(positions.numel() == y.size(0) && token_seq.numel() == y.size(0) && block_table.dim() == 2, "latent_prepare: a position and "
@@ -1363,7 +1476,14 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
     m.def("scale_into", &scale_into);
     m.def("head_norm_gate", &head_norm_gate, py::arg("o"), py::arg("y"), py::arg("gate_col"), py::arg("weight"),
           py::arg("weight_per_channel"), py::arg("eps"), py::arg("act"), py::arg("out"), py::arg("out_col"), py::arg("out_scale"),
-          py::arg("heads"), py::arg("v_dim"), py::arg("token_seq") = py::none());
+          py::arg("heads"), py::arg("v_dim"), py::arg("token_seq") = py::none(), py::arg("gate_first") = false);
+    m.def("add_normed", &add_normed, py::arg("x"), py::arg("delta"), py::arg("weight"), py::arg("eps"), py::arg("mult"), py::arg("out"),
+          py::arg("compute_dtype"));
+    m.def("causal_conv", &causal_conv, py::arg("y"), py::arg("col"), py::arg("w"), py::arg("bias"), py::arg("silu"), py::arg("tail"),
+          py::arg("cu_q"), py::arg("rows"), py::arg("tiles"), py::arg("per_tile"), py::arg("out"), py::arg("status") = py::none());
+    m.def("state_space_scan", &state_space_scan, py::arg("u"), py::arg("y"), py::arg("dt_col"), py::arg("a_log"), py::arg("dt_bias"), py::arg("d"),
+          py::arg("state"), py::arg("cu_q"), py::arg("rows"), py::arg("seqs"), py::arg("o"), py::arg("heads"), py::arg("groups"), py::arg("dim"),
+          py::arg("v_dim"), py::arg("status") = py::none());
     m.def("gla_scan", &gla_scan, py::arg("y"), py::arg("q_col"), py::arg("k_col"), py::arg("v_col"), py::arg("low_col"), py::arg("a2"),
           py::arg("a2_bias"), py::arg("inv_tau"), py::arg("q_scale"), py::arg("state"), py::arg("cu_q"), py::arg("rows"), py::arg("o"),
           py::arg("heads"), py::arg("dim"), py::arg("v_dim"), py::arg("status") = py::none(), py::arg("most_threads") = 0);
@@ -1413,10 +1533,11 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
     m.def("retention_fix", &retention_fix, py::arg("y"), py::arg("q_col"), py::arg("positions"), py::arg("frequencies"), py::arg("starts"),
           py::arg("tiles"), py::arg("decay"), py::arg("o"), py::arg("act") = 0);
     m.def("route_experts", &route_experts, py::arg("logits"), py::arg("top"), py::arg("act"), py::arg("inter"), py::arg("x") = py::none(),
-          py::arg("router") = py::none(), py::arg("mode") = 0, py::arg("scale") = 1.0, py::arg("shared_gate") = py::none());
+          py::arg("router") = py::none(), py::arg("mode") = 0, py::arg("scale") = 1.0, py::arg("shared_gate") = py::none(),
+          py::arg("bias") = py::none());
     m.def("route_topk", &route_topk, py::arg("logits"), py::arg("top"), py::arg("ids"), py::arg("weights"), py::arg("x") = py::none(),
           py::arg("router") = py::none(), py::arg("mode") = 0, py::arg("scale") = 1.0, py::arg("shared_gate") = py::none(),
-          py::arg("gates") = py::none());
+          py::arg("gates") = py::none(), py::arg("bias") = py::none());
     m.def("token_shift", &token_shift, py::arg("x"), py::arg("mu"), py::arg("state"), py::arg("cu_q"), py::arg("rows"), py::arg("token_seq"),
           py::arg("out"), py::arg("status") = py::none());
     m.def("latent_prepare", &latent_prepare, py::arg("y"), py::arg("q_col"), py::arg("q_rank"), py::arg("kv_col"), py::arg("kv_rank"),

@@ -42,6 +42,7 @@ SOURCES = [
     "attention_latent.cu",
     "latent.cu",
     "streams.cu",
+    "state_space.cu",
 ]
 HEADERS = ["common.cuh", "kernels.h", "launch.cuh", "tc_common.cuh", "gemm_epilogue.cuh", "attention_mma.cuh", "attention_decode.cuh", "attention_noalloc.h", "look_ahead.cuh"]
 

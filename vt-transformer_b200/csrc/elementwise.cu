@@ -301,6 +301,93 @@ cudaError_t launch_layernorm(int out_dtype, float* x, const void* delta, const f
                        post_eps, post_mult, stream);
 }
 
+// ------------------------------------------------------------------------- a normed result joins the stream
+
+// One block a row: x += mult * weight * d * rsqrt(mean(d^2) + eps) for the row d of a sublayer's result (a tensor, or the unadded
+// shares of a product, added in the order of their index), all in 32-bit; `out` (or null) takes the new row in the compute dtype,
+// for a sublayer that reads the stream as it is.  Without a delta the row is copied alone.  A thread keeps its first eight
+// values of d in registers; wider rows read the others again.
+template <typename T>
+__global__ void __launch_bounds__(512)
+add_normed_kernel(float* __restrict__ x, const T* __restrict__ delta, const float* __restrict__ parts, int n_parts, long long part_stride,
+                  const float* __restrict__ weight, float eps, float mult, T* __restrict__ out, int hidden) {
+    __shared__ float scratch[32];
+    pdl_launch();
+    const int first = threadIdx.x * 8;
+    float w_first[8];
+    if (weight != nullptr && first < hidden) Vec8<float>::load(weight + first, w_first);
+    pdl_wait();
+    const size_t at = (size_t)blockIdx.x * hidden;
+    auto delta_values = [&](int i, float (&d)[8]) {
+        if (delta) {
+            Vec8<T>::load(delta + at + i, d);
+            return;
+        }
+#pragma unroll
+        for (int j = 0; j < 8; ++j) d[j] = 0.f;
+#pragma unroll 4
+        for (int q = 0; q < n_parts; ++q) {
+            float e[8];
+            Vec8<float>::load(parts + at + i + q * part_stride, e);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) d[j] += e[j];
+        }
+    };
+    const bool any = delta != nullptr || parts != nullptr;
+    float d0[8], x0[8];
+    float rs = 0.f;
+    if (first < hidden) Vec8<float>::load(x + at + first, x0);
+    if (any) {
+        float ss = 0.f;
+        for (int i = first; i < hidden; i += blockDim.x * 8) {
+            float d[8];
+            delta_values(i, d);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                ss = fmaf(d[j], d[j], ss);
+                if (i == first) d0[j] = d[j];
+            }
+        }
+        rs = rsqrtf(block_sum(ss, scratch) / (float)hidden + eps) * mult;
+    }
+    for (int i = first; i < hidden; i += blockDim.x * 8) {
+        float v[8];
+        if (i == first) {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[j] = x0[j];
+        } else {
+            Vec8<float>::load(x + at + i, v);
+        }
+        if (any) {
+            float d[8], w[8];
+            if (i == first) {
+#pragma unroll
+                for (int j = 0; j < 8; ++j) { d[j] = d0[j]; w[j] = w_first[j]; }
+            } else {
+                delta_values(i, d);
+                Vec8<float>::load(weight + i, w);
+            }
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[j] += d[j] * rs * w[j];
+            Vec8<float>::store(x + at + i, v);
+        }
+        if (out) Vec8<T>::store(out + at + i, v);
+    }
+}
+
+cudaError_t launch_add_normed(int dtype, float* x, const void* delta, const float* parts, int n_parts, const float* weight, float eps, float mult,
+                              void* out, int n_tokens, int hidden, cudaStream_t stream) {
+    if (n_tokens == 0) return cudaSuccess;
+    if (hidden % 8 || (delta != nullptr && parts != nullptr) || ((delta != nullptr || parts != nullptr) && weight == nullptr)) return cudaErrorInvalidValue;
+    const int threads = min(512, max(32, ((hidden / 8 + 31) / 32) * 32));
+    const long long part_stride = (long long)n_tokens * hidden;
+    if (dtype == kBF16)
+        return launch(add_normed_kernel<__nv_bfloat16>, n_tokens, threads, 0, stream, x, (const __nv_bfloat16*)delta, parts, n_parts, part_stride,
+                      weight, eps, mult, (__nv_bfloat16*)out, hidden);
+    return launch(add_normed_kernel<float>, n_tokens, threads, 0, stream, x, (const float*)delta, parts, n_parts, part_stride, weight, eps, mult,
+                  (float*)out, hidden);
+}
+
 // ------------------------------------------------------------------------- PolyNorm
 
 // One block a row: out = a N(z) + b N(z^2) + c N(z^3) + e with N(y) = y / sqrt(mean(y^2) + eps).  Pass 1 sums z^2,

@@ -78,12 +78,13 @@ __device__ __forceinline__ void pick_top(float* z, float* w, int* picked, float*
 // dot product formed here in 32-bit: a warp an expert, a lane the same columns of every expert, the lanes' sums added by
 // the warp: the order depends on the width alone.
 // With a shared expert's gate (a vector [width], x given) z[experts] is its dot product with x, formed the same way.
+// `bias` [experts] (or null) is added to the experts' logits.
 template <typename T>
 __device__ __forceinline__ void router_logits(float* z, const float* __restrict__ logits, const T* __restrict__ x,
                                               const float* __restrict__ router, int width, int experts, int t,
-                                              const float* __restrict__ shared_gate) {
+                                              const float* __restrict__ shared_gate, const float* __restrict__ bias) {
     if (logits != nullptr)
-        for (int e = threadIdx.x; e < experts; e += blockDim.x) z[e] = logits[(size_t)t * experts + e];
+        for (int e = threadIdx.x; e < experts; e += blockDim.x) z[e] = logits[(size_t)t * experts + e] + (bias ? bias[e] : 0.f);
     if (x == nullptr) return;
     const int from = logits != nullptr ? experts : 0, rows = experts + (shared_gate != nullptr ? 1 : 0);
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
@@ -99,7 +100,7 @@ __device__ __forceinline__ void router_logits(float* z, const float* __restrict_
             for (int j = 0; j < 8; ++j) acc = fmaf(a[j], b[j], acc);
         }
         acc = warp_sum(acc);
-        if (lane == 0) z[e] = acc;
+        if (lane == 0) z[e] = acc + ((bias != nullptr && e < experts) ? bias[e] : 0.f);
     }
 }
 
@@ -108,7 +109,7 @@ template <typename T>
 __global__ void __launch_bounds__(kRouteFewThreads)
 route_experts_kernel(const float* __restrict__ logits, const T* __restrict__ x, const float* __restrict__ router, int width,
                      int experts, int top, T* __restrict__ act, int act_stride, int inter, int mode, float scale,
-                     const float* __restrict__ shared_gate) {
+                     const float* __restrict__ shared_gate, const float* __restrict__ bias) {
     __shared__ float z[kMaxExperts + 1];      // the logits (a picked one is taken out), and the shared expert's
     __shared__ float w[kMaxExperts];          // the experts' weights, zero for those not picked
     __shared__ float picked_z[kMaxExperts];
@@ -117,7 +118,7 @@ route_experts_kernel(const float* __restrict__ logits, const T* __restrict__ x, 
     pdl_wait();
     const int t = blockIdx.x, first = blockIdx.y * blockDim.x + threadIdx.x, stride = gridDim.y * blockDim.x;
     for (int e = threadIdx.x; e < experts; e += blockDim.x) w[e] = 0.f;
-    router_logits(z, logits, x, router, width, experts, t, shared_gate);
+    router_logits(z, logits, x, router, width, experts, t, shared_gate, bias);
     __syncthreads();
     pick_top(z, w, picked, picked_z, experts, top, mode, scale);
     __syncthreads();
@@ -154,14 +155,14 @@ template <typename T>
 __global__ void __launch_bounds__(kRouteThreads)
 route_topk_kernel(const float* __restrict__ logits, const T* __restrict__ x, const float* __restrict__ router, int width, int experts,
                   int top, int* __restrict__ ids, float* __restrict__ weights, int mode, float scale, const float* __restrict__ shared_gate,
-                  float* __restrict__ gates) {
+                  float* __restrict__ gates, const float* __restrict__ bias) {
     __shared__ float z[kMaxExperts + 1];
     __shared__ float picked_z[kMaxExperts];
     __shared__ int picked[kMaxExperts];
     pdl_launch();
     pdl_wait();
     const int t = blockIdx.x;
-    router_logits(z, logits, x, router, width, experts, t, shared_gate);
+    router_logits(z, logits, x, router, width, experts, t, shared_gate, bias);
     __syncthreads();
     if (shared_gate != nullptr && threadIdx.x == 0) gates[t] = 1.f / (1.f + expf(-z[experts]));
     pick_top(z, nullptr, picked, picked_z, experts, top, mode, scale);
@@ -259,15 +260,15 @@ combine_picks_kernel(const T* __restrict__ y, int width, const int* __restrict__
 
 cudaError_t launch_route_topk(int x_dtype, const float* logits, const void* x, const float* router, int width, int n_tokens, int experts,
                               int top, int* ids, float* weights, cudaStream_t stream, int mode, float scale, const float* shared_gate,
-                              float* gates) {
+                              float* gates, const float* bias) {
     if (n_tokens == 0) return cudaSuccess;
     if (experts < 1 || experts > kMaxExperts || top < 1 || top > experts || (x != nullptr && width % 8)) return cudaErrorInvalidValue;
     if (shared_gate != nullptr && (x == nullptr || gates == nullptr)) return cudaErrorInvalidValue;
     if (x_dtype == kBF16)
         return launch(route_topk_kernel<__nv_bfloat16>, n_tokens, kRouteThreads, 0, stream, logits, (const __nv_bfloat16*)x, router, width,
-                      experts, top, ids, weights, mode, scale, shared_gate, gates);
+                      experts, top, ids, weights, mode, scale, shared_gate, gates, bias);
     return launch(route_topk_kernel<float>, n_tokens, kRouteThreads, 0, stream, logits, (const float*)x, router, width, experts, top, ids,
-                  weights, mode, scale, shared_gate, gates);
+                  weights, mode, scale, shared_gate, gates, bias);
 }
 
 cudaError_t launch_expert_lists(const int* ids, int n_picks, int experts, int list_stride, int* lists, int* counts, cudaStream_t stream) {
@@ -299,7 +300,7 @@ cudaError_t launch_combine_picks(int dtype, const void* y, int width, const int*
 
 cudaError_t launch_route_experts(int dtype, const float* logits, const void* x, const float* router, int width, int n_tokens, int experts,
                                  int top, void* act, int act_stride, int inter, cudaStream_t stream, int mode, float scale,
-                                 const float* shared_gate) {
+                                 const float* shared_gate, const float* bias) {
     if (n_tokens == 0) return cudaSuccess;
     if (shared_gate != nullptr && x == nullptr) return cudaErrorInvalidValue;
     if (experts < 1 || experts > kMaxExperts || top < 1 || top > experts || (x != nullptr && width % 8)) return cudaErrorInvalidValue;
@@ -308,9 +309,9 @@ cudaError_t launch_route_experts(int dtype, const float* logits, const void* x, 
     const dim3 grid(n_tokens, few ? max(1, min(min(4, 296 / n_tokens), act_stride / (8 * threads))) : 1);
     if (dtype == kBF16)
         return launch(route_experts_kernel<__nv_bfloat16>, grid, threads, 0, stream, logits, (const __nv_bfloat16*)x, router, width,
-                      experts, top, (__nv_bfloat16*)act, act_stride, inter, mode, scale, shared_gate);
+                      experts, top, (__nv_bfloat16*)act, act_stride, inter, mode, scale, shared_gate, bias);
     return launch(route_experts_kernel<float>, grid, threads, 0, stream, logits, (const float*)x, router, width, experts, top,
-                  (float*)act, act_stride, inter, mode, scale, shared_gate);
+                  (float*)act, act_stride, inter, mode, scale, shared_gate, bias);
 }
 
 }  // namespace vtb

@@ -56,7 +56,29 @@ cudaError_t launch_delta_scan(int dtype, const void* y, int stride, int r_col, i
 // of padding tokens (< 0) become zero.
 cudaError_t launch_head_norm_gate(int dtype, const float* o, const void* y, int y_stride, int gate_col, const float* weight,
                                   int weight_per_channel, float eps, int act, void* out, int out_stride, int out_col,
-                                  float out_scale, const int* token_seq, int n_tokens, int heads, int v_dim, cudaStream_t stream);
+                                  float out_scale, const int* token_seq, int n_tokens, int heads, int v_dim, cudaStream_t stream,
+                                  int gate_first = 0);
+// (gate_first: the gate multiplies o before the norm)
+
+// x += mult * weight * d * rsqrt(mean(d^2) + eps) row by row, d = delta (of the compute dtype) or the sum of parts
+// [n_parts, n_tokens, hidden]; out (or null) takes the new rows in the compute dtype; without d the rows are copied alone.
+cudaError_t launch_add_normed(int dtype, float* x, const void* delta, const float* parts, int n_parts, const float* weight, float eps, float mult,
+                              void* out, int n_tokens, int hidden, cudaStream_t stream);
+
+// State-space mixers (state_space.cu).  The convolution: out[t, c] = act(bias[c] + sum_j w[j, c] y[t - taps + 1 + j, col + c]) for
+// w [taps, channels], act 1 silu, 0 nothing; the rows before a sequence's first token of the step from tail [state_rows, taps - 1,
+// channels] (oldest first), which is renewed; tiles [n_tiles, 2] (sequence, first of its new tokens) of per_tile >= taps - 1 tokens,
+// or null: tile = sequence.
+cudaError_t launch_causal_conv(int dtype, const void* y, int stride, int col, int channels, const float* w, int taps, const float* bias, int act,
+                               float* tail, int state_rows, const int* cu_q, const int* seq_rows, int n_seqs, const int* tiles, int n_tiles,
+                               int per_tile, void* out, int* status, cudaStream_t stream);
+// The recurrence token by token: u [tokens, u_stride] holds x [heads * v_dim], B [groups * dim] and C [groups * dim] side by side, the
+// raw step sizes are y[t, dt_col + h]; with d = softplus(raw + dt_bias[h]): S <- exp(-exp(a_log[h]) d) S + d B x^T, out = S^T C + d_skip[h] x,
+// head h with group h / (heads / groups).  state [state_rows, heads, dim, v_dim]; seqs [n_listed]: the step's sequences that run here (null: all).
+cudaError_t launch_state_space_scan(int dtype, const void* u, int u_stride, const void* y, int stride, int dt_col, const float* a_log,
+                                    const float* dt_bias, const float* d, float* state, int state_rows, const int* cu_q, const int* rows,
+                                    int n_seqs, const int* seqs, int n_listed, float* out, int heads, int groups, int dim, int v_dim, int* status,
+                                    cudaStream_t stream);
 
 // Recurrences with one decay a head (recurrent_gated.cu), in the manner of the scans above: q, k, v and the gates' inputs are
 // columns of y; the state is read at rows[sequence] and left as after the sequence's last token; out [tokens, heads * v_dim].
@@ -167,13 +189,13 @@ cudaError_t launch_retention_fix(int dtype, const void* y, int stride, int q_col
 // multiplied by sigmoid(x[t, :] . shared_gate); route_topk leaves that number in gates[t], combine_picks multiplies shared_y by it.
 cudaError_t launch_route_experts(int dtype, const float* logits, const void* x, const float* router, int width, int n_tokens, int experts,
                                  int top, void* act, int act_stride, int inter, cudaStream_t stream, int mode = 0, float scale = 1.f,
-                                 const float* shared_gate = nullptr);
+                                 const float* shared_gate = nullptr, const float* bias = nullptr);
 // The grouped form: ids / weights [n_tokens, top] of each token's picks; lists [experts, list_stride] of the picks (flat
 // index t * top + k) of every expert in rising order and counts [experts]; sorted [n_picks, width] the input rows by
 // expert and where [n_picks] each pick's row; out[t] = sum_k weights[t, k] * y[where[t * top + k]] (+ shared_y[t]).
 cudaError_t launch_route_topk(int x_dtype, const float* logits, const void* x, const float* router, int width, int n_tokens, int experts,
                               int top, int* ids, float* weights, cudaStream_t stream, int mode = 0, float scale = 1.f,
-                              const float* shared_gate = nullptr, float* gates = nullptr);
+                              const float* shared_gate = nullptr, float* gates = nullptr, const float* bias = nullptr);
 cudaError_t launch_expert_lists(const int* ids, int n_picks, int experts, int list_stride, int* lists, int* counts, cudaStream_t stream);
 cudaError_t launch_gather_picks(int dtype, const void* x, int width, const int* lists, int list_stride, const int* counts, int experts,
                                 int top, int n_picks, void* sorted, int* where, cudaStream_t stream);

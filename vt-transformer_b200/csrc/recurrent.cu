@@ -550,8 +550,15 @@ cudaError_t launch_retention_fix(int dtype, const void* y, int stride, int q_col
 
 // ------------------------------------------------------------------------- norm of each head's output, gate
 
-// One warp for a (token, head): out = out_scale * o / sqrt(mean(o^2) + eps) * w * act(gate), all in 32-bit.
-template <typename T>
+// v act(z): act 0 silu, 1 sigmoid.
+__device__ __forceinline__ float gated(float v, float z, int act) {
+    const float s = 1.f / (1.f + expf(-z));
+    return v * (act == 0 ? z * s : s);
+}
+
+// One warp for a (token, head): out = out_scale * o / sqrt(mean(o^2) + eps) * w * act(gate), all in 32-bit.  GATE_FIRST: the gate
+// multiplies o before the norm, v = o act(gate), out = out_scale * v / sqrt(mean(v^2) + eps) * w.
+template <typename T, bool GATE_FIRST>
 __global__ void __launch_bounds__(128)
 head_norm_gate_kernel(const float* __restrict__ o, const T* __restrict__ y, int y_stride, int gate_col,
                       const float* __restrict__ weight, int weight_per_channel, float eps, int act, T* __restrict__ out,
@@ -569,13 +576,20 @@ head_norm_gate_kernel(const float* __restrict__ o, const T* __restrict__ y, int 
         return;
     }
     const float* src = o + ((size_t)t * heads + h) * v_dim;
+    const T* gate = y + (size_t)t * y_stride + gate_col + h * v_dim;
     float ss = 0.f;
-    for (int i = lane; i < v_dim; i += 32) ss = fmaf(src[i], src[i], ss);
+    for (int i = lane; i < v_dim; i += 32) {
+        const float v = GATE_FIRST ? gated(src[i], to_float(gate[i]), act) : src[i];
+        ss = fmaf(v, v, ss);
+    }
     ss = warp_sum(ss);
     const float r = rsqrtf(ss / (float)v_dim + eps) * out_scale;
-    const T* gate = y + (size_t)t * y_stride + gate_col + h * v_dim;
     const float* w = weight + (weight_per_channel ? h * v_dim : 0);
     for (int i = lane; i < v_dim; i += 32) {
+        if (GATE_FIRST) {
+            dst[i] = from_float<T>(gated(src[i], to_float(gate[i]), act) * r * w[i]);
+            continue;
+        }
         const float z = to_float(gate[i]);
         const float s = 1.f / (1.f + expf(-z));
         dst[i] = from_float<T>(src[i] * r * w[i] * (act == 0 ? z * s : s));
@@ -584,7 +598,7 @@ head_norm_gate_kernel(const float* __restrict__ o, const T* __restrict__ y, int 
 
 // The same for heads of many values (heads normed together are one head as wide as all of them): a CTA a (token, head),
 // its warps' sums of squares added in the order of the warps.
-template <typename T>
+template <typename T, bool GATE_FIRST>
 __global__ void __launch_bounds__(256)
 head_norm_gate_wide_kernel(const float* __restrict__ o, const T* __restrict__ y, int y_stride, int gate_col,
                            const float* __restrict__ weight, int weight_per_channel, float eps, int act, T* __restrict__ out,
@@ -599,8 +613,12 @@ head_norm_gate_wide_kernel(const float* __restrict__ o, const T* __restrict__ y,
         return;
     }
     const float* src = o + ((size_t)t * heads + h) * v_dim;
+    const T* gate = y + (size_t)t * y_stride + gate_col + h * v_dim;
     float ss = 0.f;
-    for (int i = threadIdx.x; i < v_dim; i += 256) ss = fmaf(src[i], src[i], ss);
+    for (int i = threadIdx.x; i < v_dim; i += 256) {
+        const float v = GATE_FIRST ? gated(src[i], to_float(gate[i]), act) : src[i];
+        ss = fmaf(v, v, ss);
+    }
     ss = warp_sum(ss);
     if ((threadIdx.x & 31) == 0) sums[threadIdx.x >> 5] = ss;
     __syncthreads();
@@ -608,35 +626,39 @@ head_norm_gate_wide_kernel(const float* __restrict__ o, const T* __restrict__ y,
 #pragma unroll
     for (int k = 0; k < 8; ++k) total += sums[k];
     const float r = rsqrtf(total / (float)v_dim + eps) * out_scale;
-    const T* gate = y + (size_t)t * y_stride + gate_col + h * v_dim;
     const float* w = weight + (weight_per_channel ? h * v_dim : 0);
     for (int i = threadIdx.x; i < v_dim; i += 256) {
+        if (GATE_FIRST) {
+            dst[i] = from_float<T>(gated(src[i], to_float(gate[i]), act) * r * w[i]);
+            continue;
+        }
         const float z = to_float(gate[i]);
         const float sg = 1.f / (1.f + expf(-z));
         dst[i] = from_float<T>(src[i] * r * w[i] * (act == 0 ? z * sg : sg));
     }
 }
 
+template <typename T, bool GATE_FIRST>
+static cudaError_t launch_head_norm_gate_t(const float* o, const void* y, int y_stride, int gate_col, const float* weight, int weight_per_channel,
+                                           float eps, int act, void* out, int out_stride, int out_col, float out_scale, const int* token_seq,
+                                           int n_tokens, int heads, int v_dim, cudaStream_t stream) {
+    const long long pairs = (long long)n_tokens * heads;
+    if (v_dim >= 1024)
+        return launch(head_norm_gate_wide_kernel<T, GATE_FIRST>, (int)pairs, 256, 0, stream, o, (const T*)y, y_stride, gate_col, weight,
+                      weight_per_channel, eps, act, (T*)out, out_stride, out_col, out_scale, token_seq, heads, v_dim);
+    return launch(head_norm_gate_kernel<T, GATE_FIRST>, (int)((pairs + 3) / 4), 128, 0, stream, o, (const T*)y, y_stride, gate_col, weight,
+                  weight_per_channel, eps, act, (T*)out, out_stride, out_col, out_scale, token_seq, n_tokens, heads, v_dim);
+}
+
 cudaError_t launch_head_norm_gate(int dtype, const float* o, const void* y, int y_stride, int gate_col, const float* weight,
                                   int weight_per_channel, float eps, int act, void* out, int out_stride, int out_col,
-                                  float out_scale, const int* token_seq, int n_tokens, int heads, int v_dim, cudaStream_t stream) {
-    const long long pairs = (long long)n_tokens * heads;
-    if (pairs == 0) return cudaSuccess;
-    if (v_dim >= 1024) {
-        if (dtype == kBF16)
-            return launch(head_norm_gate_wide_kernel<__nv_bfloat16>, (int)pairs, 256, 0, stream, o, (const __nv_bfloat16*)y, y_stride,
-                          gate_col, weight, weight_per_channel, eps, act, (__nv_bfloat16*)out, out_stride, out_col, out_scale, token_seq,
-                          heads, v_dim);
-        return launch(head_norm_gate_wide_kernel<float>, (int)pairs, 256, 0, stream, o, (const float*)y, y_stride, gate_col, weight,
-                      weight_per_channel, eps, act, (float*)out, out_stride, out_col, out_scale, token_seq, heads, v_dim);
-    }
-    const int blocks = (int)((pairs + 3) / 4);
-    if (dtype == kBF16)
-        return launch(head_norm_gate_kernel<__nv_bfloat16>, blocks, 128, 0, stream, o, (const __nv_bfloat16*)y, y_stride, gate_col,
-                      weight, weight_per_channel, eps, act, (__nv_bfloat16*)out, out_stride, out_col, out_scale, token_seq,
-                      n_tokens, heads, v_dim);
-    return launch(head_norm_gate_kernel<float>, blocks, 128, 0, stream, o, (const float*)y, y_stride, gate_col, weight,
-                  weight_per_channel, eps, act, (float*)out, out_stride, out_col, out_scale, token_seq, n_tokens, heads, v_dim);
+                                  float out_scale, const int* token_seq, int n_tokens, int heads, int v_dim, cudaStream_t stream,
+                                  int gate_first) {
+    if ((long long)n_tokens * heads == 0) return cudaSuccess;
+    auto run = dtype == kBF16 ? (gate_first ? launch_head_norm_gate_t<__nv_bfloat16, true> : launch_head_norm_gate_t<__nv_bfloat16, false>)
+                              : (gate_first ? launch_head_norm_gate_t<float, true> : launch_head_norm_gate_t<float, false>);
+    return run(o, y, y_stride, gate_col, weight, weight_per_channel, eps, act, out, out_stride, out_col, out_scale, token_seq, n_tokens, heads,
+               v_dim, stream);
 }
 
 }  // namespace vtb

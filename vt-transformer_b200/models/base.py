@@ -6,7 +6,7 @@ from typing import Dict, Optional
 
 import torch
 
-from ..parts.base import CacheView, ParamSpec, ResidualStream, Runtime, StreamBundle, build_part
+from ..parts.base import CacheView, ParamSpec, ResidualStream, Runtime, StreamBundle, build_part, join_cache_specs
 from ..parts.specs import ModelSpec
 from ..weights.loader import WeightSource, check_against, load_report
 
@@ -17,7 +17,7 @@ class DecoderModel:
 
     ``order`` is data: ``spec.order[n] = RunSpec(block, cache, writes)``.  The cache slots
     that the runs name are declared by ``cache_slots()``: slot id -> the cache spec of the
-    block whose run writes it."""
+    block whose run writes it, under the widest window of the runs that read it."""
 
     def __init__(self, spec: ModelSpec, rt: Runtime):
         self.spec = spec
@@ -52,10 +52,10 @@ class DecoderModel:
                 else:
                     if slot not in slots:
                         raise ValueError(f"run {n} reads cache slot {slot} before any run wrote it")
-                    have = slots[slot]
-                    if type(have) is not type(spec) or getattr(have, "kv_heads", None) != getattr(spec, "kv_heads", None) \
-                            or getattr(have, "head_dim", None) != getattr(spec, "head_dim", None):
-                        raise ValueError(f"run {n}: cache slot {slot} has another layout than block {run.block} reads")
+                    try:
+                        slots[slot] = join_cache_specs(slots[slot], spec)
+                    except ValueError:
+                        raise ValueError(f"run {n}: cache slot {slot} has another layout than block {run.block} reads") from None
         need = self.embedding.cache_spec()
         if need is not None:
             slot = self.spec.embedding_cache

@@ -136,14 +136,16 @@ def polynorm(z: torch.Tensor, coefficients: torch.Tensor, eps: float, out: torch
 
 def head_norm_gate(o: torch.Tensor, y: torch.Tensor, gate_col: int, weight: torch.Tensor, weight_per_channel: bool,
                    eps: float, act: str, out: torch.Tensor, out_col: int, out_scale: float, heads: int, v_dim: int,
-                   token_seq: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   token_seq: Optional[torch.Tensor] = None, gate_first: bool = False) -> torch.Tensor:
     """out[t, out_col + h * v_dim + i] = out_scale * o[t, h, i] / sqrt(mean_i(o[t, h, :]^2) + eps) * w * act(gate)
     for the 32-bit o [T, heads * v_dim] of a recurrent mixer; gate = y[t, gate_col + h * v_dim + i]; w = weight[i]
     (a weight [v_dim] shared by the heads) or, with ``weight_per_channel``, weight[h * v_dim + i]; ``act`` is
     "silu" or "sigmoid".  32-bit until the one rounding into ``out``.  With ``token_seq`` (the step's sequence index
-    of every token) the rows of padding tokens (-1), for which nothing ran, become zero."""
-    backend().head_norm_gate(o, y, int(gate_col), weight, bool(weight_per_channel), float(eps), _GATE_ACTS[act], out,
-                             int(out_col), float(out_scale), int(heads), int(v_dim), token_seq)
+    of every token) the rows of padding tokens (-1), for which nothing ran, become zero.  ``gate_first``: act(gate) multiplies
+    o before its norm, not after."""
+    args = (o, y, int(gate_col), weight, bool(weight_per_channel), float(eps), _GATE_ACTS[act], out, int(out_col), float(out_scale),
+            int(heads), int(v_dim), token_seq)
+    backend().head_norm_gate(*args, gate_first=True) if gate_first else backend().head_norm_gate(*args)
     return out
 
 
@@ -276,6 +278,42 @@ def retention_scan(y, q_col: int, k_col: int, v_col: int, decay: torch.Tensor, k
     return o
 
 
+def add_normed(x: torch.Tensor, delta, post, out: Optional[torch.Tensor], dtype) -> torch.Tensor:
+    """x += m * w * delta / sqrt(mean(delta^2) + e) row by row with ``post`` = (w [H] float32, e, m), in 32-bit, and ``out`` (None:
+    nothing) takes the new rows in the compute dtype ``dtype``.  ``delta``: a tensor of that dtype, a ``SplitSum``, or None (the
+    rows are copied alone)."""
+    if isinstance(delta, SplitSum):
+        delta = delta.shares
+    weight, eps, mult = post if delta is not None else (None, 0.0, 1.0)
+    backend().add_normed(x, delta, weight, float(eps), float(mult), out, 1 if dtype == torch.bfloat16 else 0)
+    return x
+
+
+CAUSAL_CONV_TILE = 16            # tokens that a CTA of the convolution over a step's tokens walks (the most taps have 15 before them)
+
+
+def causal_conv(y, col: int, w: torch.Tensor, bias, tail, ctx, out: torch.Tensor, silu: bool = True, status=None) -> torch.Tensor:
+    """out[t, c] = act(bias[c] + sum_j w[j, c] y[t - taps + 1 + j, col + c]) for w [taps, channels] float32 (the last tap the present
+    token's) and act silu or nothing; taps added oldest first in 32-bit.  The rows before a sequence's first token of the step come
+    from ``tail`` [request rows, taps - 1, channels] (float32, oldest first, zeros at admission; None with one tap), which then
+    holds the sequence's last taps - 1 inputs."""
+    tiles = None if ctx.max_q_len == 1 and ctx.n_tokens == ctx.n_seqs else _attention_tiles(ctx, CAUSAL_CONV_TILE, y.device)
+    backend().causal_conv(y, int(col), w, bias, bool(silu), tail, ctx.cu_q, ctx.rows, tiles, CAUSAL_CONV_TILE, out, status)
+    return out
+
+
+def state_space(u, y, dt_col: int, a_log, dt_bias, d, state: torch.Tensor, ctx, o: torch.Tensor, heads: int, groups: int, dim: int,
+                v_dim: int, status=None) -> torch.Tensor:
+    """A state-space recurrence over the step's tokens, sequence by sequence and head by head.  ``u`` [T, heads * v_dim +
+    2 groups * dim] holds x, B and C side by side; the raw step size of head h is y[t, dt_col + h].  With s = softplus(raw + dt_bias[h]):
+    S <- exp(-exp(a_log[h]) s) S + s B x^T, o = S^T C + d[h] x, head h with group h // (heads / groups).  ``state`` [request rows,
+    heads, dim, v_dim] float32 is read at the step's ``ctx.rows`` and left as after the last token; ``o`` [T, heads * v_dim] float32.
+    Step sizes, decays, state and sums in 32-bit."""
+    backend().state_space_scan(u, y, int(dt_col), a_log, dt_bias, d, state, ctx.cu_q, ctx.rows, None, o, int(heads), int(groups), int(dim),
+                               int(v_dim), status)
+    return o
+
+
 def attention_prepare(y, q_col: int, k_col: int, v_col: int, ctx, frequencies, norm_eps, k_cache, v_cache, block_table,
                       heads: int, kv_heads: int, dim: int, v_dim: int, store: bool = True, status=None, v_heads=None,
                       q_weight=None, k_weight=None, norm_first: bool = False, whole_projection: bool = False,
@@ -391,19 +429,20 @@ _ROUTER_WEIGHTS = {"softmax": 0, "sigmoid_share": 1}
 
 
 def route_topk(logits, top: int, ids: torch.Tensor, weights: torch.Tensor, x=None, router=None, weights_by: str = "softmax",
-               scale: float = 1.0, shared_gate=None, gates=None) -> None:
+               scale: float = 1.0, shared_gate=None, gates=None, bias=None) -> None:
     """ids[t, k] and weights[t, k]: the ``top`` largest router logits of every token in falling order (the lower index
     among equals) and the softmax over them (which is the softmax over all logits, divided by the picks' sum of it), times
     ``scale``.  ``logits`` [tokens, experts] float32, or None with the tokens' input rows
     ``x`` [tokens, width] and the router's matrix ``router`` [experts, width] (float32), from which the kernel forms
     them as 32-bit dot products.  ``weights_by`` "sigmoid_share": a pick weighs as sigmoid(logit) over the picks' sum of
     them (+ 1e-20), times ``scale``.  ``shared_gate`` [width] float32 (with ``x``): gates[t] = sigmoid(x[t] . shared_gate), in
-    32-bit."""
+    32-bit.  ``bias`` [experts] float32 is added to the logits."""
     args = (logits, int(top), ids, weights, x, router, _ROUTER_WEIGHTS[weights_by], float(scale))
+    extra = {} if bias is None else {"bias": bias}
     if shared_gate is None:
-        backend().route_topk(*args)
+        backend().route_topk(*args, **extra)
     else:
-        backend().route_topk(*args, shared_gate, gates)
+        backend().route_topk(*args, shared_gate, gates, **extra)
 
 
 def expert_lists(ids: torch.Tensor, lists: torch.Tensor, counts: torch.Tensor) -> None:
@@ -504,18 +543,20 @@ def attention_latent(q, q_col: int, out, out_col: int, pages, ctx, block_table, 
 
 
 def route_experts(logits, top: int, act: torch.Tensor, inter: int, x=None, router=None, weights_by: str = "softmax",
-                  scale: float = 1.0, shared_gate=None) -> torch.Tensor:
+                  scale: float = 1.0, shared_gate=None, bias=None) -> torch.Tensor:
     """For every token (row): the ``top`` largest of its router logits [experts] (float32; the lower index among
     equals) choose its experts, the softmax over the chosen logits weighs them; columns [e * inter, (e + 1) * inter) of
     ``act`` (what expert e's last product multiplies) are multiplied by expert e's weight, and set to zero for an
     expert that was not chosen.  Columns beyond experts * inter (an expert that every token uses) stay.  ``logits`` may be
     None with ``x`` and ``router`` given, and ``weights_by`` and ``scale``, as for ``route_topk``.  ``shared_gate`` [width]
-    float32 (with ``x``): the columns beyond are multiplied by sigmoid(x[t] . shared_gate), formed in 32-bit."""
+    float32 (with ``x``): the columns beyond are multiplied by sigmoid(x[t] . shared_gate), formed in 32-bit.  ``bias`` [experts]
+    float32 is added to the logits."""
     args = (logits, int(top), act, int(inter), x, router, _ROUTER_WEIGHTS[weights_by], float(scale))
+    extra = {} if bias is None else {"bias": bias}
     if shared_gate is None:
-        backend().route_experts(*args)
+        backend().route_experts(*args, **extra)
     else:
-        backend().route_experts(*args, shared_gate)
+        backend().route_experts(*args, shared_gate, **extra)
     return act
 
 
@@ -1133,6 +1174,6 @@ def _counted(fn):
     return wrapper
 
 
-for _name in ("embedding_pair", "streams_norm", "relu_square", "gate_into", "gated_delta_scan", "conv_tail_update", "memory_scan", "normed_sum", "add_rows", "embedding", "logits_scale_cap", "rmsnorm", "layernorm", "polynorm", "scale_into", "head_norm_gate", "gla_scan", "delta_scan", "retention_scan", "route_experts", "attention_differential", "route_topk", "expert_lists", "gather_picks", "combine_picks",
+for _name in ("add_normed", "causal_conv", "state_space", "embedding_pair", "streams_norm", "relu_square", "gate_into", "gated_delta_scan", "conv_tail_update", "memory_scan", "normed_sum", "add_rows", "embedding", "logits_scale_cap", "rmsnorm", "layernorm", "polynorm", "scale_into", "head_norm_gate", "gla_scan", "delta_scan", "retention_scan", "route_experts", "attention_differential", "route_topk", "expert_lists", "gather_picks", "combine_picks",
               "token_shift", "latent_prepare", "head_matmul", "attention_latent", "xielu", "gate_clamp", "attention_prepare", "attention_general", "silu_mul", "rope_store", "linear", "paged_attention", "argmax", "sample"):  # the others count where they launch
     globals()[_name] = _counted(globals()[_name])

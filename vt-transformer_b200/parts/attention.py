@@ -14,7 +14,7 @@ def _attention(spec, prefix, rt):
     values as wide as keys and a causal or windowed mask; everything else runs ``GeneralAttention``."""
     plain = (spec.v_dim in (None, spec.head_dim) and spec.qk_norm_eps is None and spec.chunk is None
              and spec.position.kind != "rotary_computed" and not spec.keep_first and spec.proj_norm_eps is None
-             and spec.q_temp is None and spec.softcap is None and spec.sink == "none" and spec.gate == "none"
+             and spec.head_norm_eps is None and not spec.values_from_keys and spec.q_temp is None and spec.softcap is None and spec.sink == "none" and spec.gate == "none"
              and spec.weight_suffix == ".weight" and spec.bias_suffix == ".bias")
     return (PagedAttention if plain else GeneralAttention)(spec, prefix, rt)
 
@@ -107,7 +107,8 @@ class GeneralAttention(ProjectedMixer):
     than keys (``v_dim``), a rotation of the first dimensions of a head only, with the angle formed where it is used
     (``rotary_computed``), q and k divided by their root mean square after the rotation (``qk_norm_eps``), and a mask
     of chunks (``chunk``) beside or instead of the window; a norm of q and of k over all their heads together with a
-    weight, before the rotation (``proj_norm_eps``); a query temperature that grows with the position (``q_temp``); capped
+    weight, before the rotation (``proj_norm_eps``), or of every head by itself with a weight its heads share (``head_norm_eps``);
+    values that are the keys' projections (``values_from_keys``); a query temperature that grows with the position (``q_temp``); capped
     scores (``softcap``); a sink in the softmax's denominator (``sink``); a gate on the heads' results, one number a head
     or one an element, whose matrix joins the packed input product (``gate``); biases.  One kernel norms, rotates and
     scales q and k (32-bit) and stores k and v into the pages; the attention kernel walks the visible keys of every
@@ -119,8 +120,10 @@ class GeneralAttention(ProjectedMixer):
             raise ValueError(f"attention: sink '{spec.sink}' is not known; known: none, zero, learned")
         if spec.gate not in ("none", "head", "element"):
             raise ValueError(f"attention: gate '{spec.gate}' is not known; known: none, head, element")
-        if spec.proj_norm_eps is not None and spec.qk_norm_eps is not None:
-            raise ValueError("attention: a norm of q and k over the whole projection or head by head, not both")
+        if sum(e is not None for e in (spec.proj_norm_eps, spec.qk_norm_eps, spec.head_norm_eps)) > 1:
+            raise ValueError("attention: one norm of q and k: over the whole projection, or head by head before or after the rotation")
+        if spec.values_from_keys and spec.v_dim not in (None, spec.head_dim):
+            raise ValueError("attention: values that are the keys' projections are as wide as keys")
         if spec.position.kind not in ("rotary_computed", "none"):
             raise ValueError(f"attention: position encoding '{spec.position.kind}' is not built beside the general options; "
                              f"known: rotary_computed, none")
@@ -140,6 +143,8 @@ class GeneralAttention(ProjectedMixer):
         s, p, x, bx = self.spec, self.prefix, self.spec.weight_suffix, self.spec.bias_suffix
         q, k, v, o = s.names
         sizes = {q: s.heads * s.head_dim, k: s.kv_heads * s.head_dim, v: s.kv_heads * self.v_dim}
+        if s.values_from_keys:
+            del sizes[v]
         out = {f"{p}{n}{x}": ParamSpec((size, s.hidden)) for n, size in sizes.items()}
         out[f"{p}{o}{x}"] = ParamSpec((s.hidden, s.heads * self.v_dim))
         if s.qkv_bias:
@@ -149,6 +154,8 @@ class GeneralAttention(ProjectedMixer):
         if s.proj_norm_eps is not None:
             out[p + s.norm_names[0]] = ParamSpec((sizes[q],), role="vector", init="one_plus_normal")
             out[p + s.norm_names[1]] = ParamSpec((sizes[k],), role="vector", init="one_plus_normal")
+        if s.head_norm_eps is not None:
+            out.update({p + n: ParamSpec((s.head_dim,), role="vector", init="one_plus_normal") for n in s.norm_names})
         if s.sink == "learned":
             out[p + s.sink_name] = ParamSpec((s.heads,), role="vector")
         if s.gate != "none":
@@ -158,15 +165,16 @@ class GeneralAttention(ProjectedMixer):
     def load(self, get) -> None:
         s, p, rt, x, bx = self.spec, self.prefix, self.rt, self.spec.weight_suffix, self.spec.bias_suffix
         q, k, v, o = s.names
-        self._in = [rt.param(get(f"{p}{n}{x}")) for n in (q, k, v)]
-        self._in_bias = [rt.param(get(f"{p}{n}{bx}"), "vector") for n in (q, k, v)] if s.qkv_bias else [None, None, None]
+        own = (q, k) if s.values_from_keys else (q, k, v)
+        self._in = [rt.param(get(f"{p}{n}{x}")) for n in own]
+        self._in_bias = [rt.param(get(f"{p}{n}{bx}"), "vector") if s.qkv_bias else None for n in own]
         if s.gate != "none":
             self._in.append(rt.param(get(p + s.gate_name)))
             self._in_bias.append(None)
         self.w_o = rt.param(get(f"{p}{o}{x}"))
         self.b_o = rt.param(get(f"{p}{o}{bx}"), "vector") if s.out_bias else None
         self.q_weight = self.k_weight = None
-        if s.proj_norm_eps is not None:
+        if s.proj_norm_eps is not None or s.head_norm_eps is not None:
             self.q_weight = rt.param(get(p + s.norm_names[0]), "vector")
             self.k_weight = rt.param(get(p + s.norm_names[1]), "vector")
         self.sinks = None
@@ -202,12 +210,15 @@ class GeneralAttention(ProjectedMixer):
         s, ops = self.spec, self.rt.ops
         freq = getattr(self.position, "frequencies", None)
         k_pages, v_pages = cache.pages["k"], cache.pages["v"]
-        whole = s.proj_norm_eps is not None
-        ops.attention_prepare(y, cols[0], cols[1], cols[2], ctx, freq, s.proj_norm_eps if whole else s.qk_norm_eps, k_pages, v_pages,
+        whole, each = s.proj_norm_eps is not None, s.head_norm_eps is not None
+        eps = s.proj_norm_eps if whole else (s.head_norm_eps if each else s.qk_norm_eps)
+        # (values that are the keys' projections are read where the keys' lie: the kernel leaves those as they are)
+        ops.attention_prepare(y, cols[0], cols[1], cols[1] if s.values_from_keys else cols[2], ctx, freq, eps, k_pages, v_pages,
                               cache.block_table, s.heads, s.kv_heads, s.head_dim, self.v_dim, store=cache.writes, status=ctx.status,
-                              q_weight=self.q_weight, k_weight=self.k_weight, norm_first=whole, whole_projection=whole,
+                              q_weight=self.q_weight, k_weight=self.k_weight, norm_first=whole or each, whole_projection=whole,
                               rot_mult=getattr(self.position, "mult", 1.0), q_temp=s.q_temp)
         gated = s.gate != "none"
+        gate_col = cols[-1] if gated else 0
         extras = s.softcap is not None or self.sinks is not None
         takes = ops.tensor_core_attention_takes_extras if extras else ops.tensor_core_attention_takes
         if cols[0] == 0 and not s.keep_first and takes(y.dtype, s.heads, s.kv_heads, s.head_dim, self.v_dim, cache.page_size):
@@ -221,14 +232,14 @@ class GeneralAttention(ProjectedMixer):
             ops.paged_attention(y, o, k_pages, v_pages, ctx, cache.block_table, s.heads, s.kv_heads, s.head_dim, s.window,
                                 self.scale, status=ctx.status, chunk=s.chunk, sinks=self.sinks, softcap=s.softcap)
             if gated:
-                ops.gate_into(o, y, cols[3], s.gate, out, out_col, out_scale, s.heads, self.v_dim)
+                ops.gate_into(o, y, gate_col, s.gate, out, out_col, out_scale, s.heads, self.v_dim)
             elif not direct:
                 ops.scale_into(o, out, out_col, out_scale)
             return
         ops.attention_general(y, cols[0], out, out_col, out_scale, k_pages, v_pages, ctx, cache.block_table, s.heads,
                               s.kv_heads, s.head_dim, self.v_dim, s.window, s.chunk, self.scale, status=ctx.status,
                               keep_first=s.keep_first if s.window else 0, sinks=self.sinks, softcap=s.softcap,
-                              gate=s.gate, gate_col=cols[3] if s.gate != "none" else 0)
+                              gate=s.gate, gate_col=gate_col)
 
 
 @register_part("mixer", "differential_attention")

@@ -173,6 +173,21 @@ register_cache_kind(LatentCacheSpec, lambda s: PagedLayout((("c", 1, s.width),),
 register_cache_kind(StateSpec, lambda s: StateLayout(tuple(s.shape), s.dtype))
 
 
+def join_cache_specs(have, spec):
+    """The cache spec under which a slot serves a run that wrote it with ``have`` and one that reads it with ``spec``: the same
+    layout, the wider of the two windows.  Raises ValueError where they differ in anything else."""
+    import dataclasses
+    open_ended = {n: v for n, v in (("window", None), ("keep_first", 0)) if hasattr(have, n)}
+    if type(have) is not type(spec) or dataclasses.replace(have, **open_ended) != dataclasses.replace(spec, **open_ended):
+        raise ValueError("another layout")
+    if "window" not in open_ended or have.window is None:
+        return have
+    wide = {"window": None if spec.window is None else max(have.window, spec.window)}
+    if "keep_first" in open_ended:
+        wide["keep_first"] = 0 if wide["window"] is None else max(have.keep_first, spec.keep_first)
+    return dataclasses.replace(have, **wide)
+
+
 @dataclass
 class CacheView:
     """What one run of a block sees of the cache.
@@ -354,6 +369,19 @@ class ResidualStream:
         if not getattr(norm, "takes_post", False):
             raise RuntimeError(f"norm '{norm.spec.kind}' cannot add a delta that is normed first")
         return norm(self.x, delta=delta, rows=rows, status=self.status, post=post)
+
+    def plain(self, rt) -> torch.Tensor:
+        """The stream as it is, in the compute dtype, for a sublayer that reads it without a norm.  A pending result (which must
+        be one that is normed before it is added) joins the stream in the same pass."""
+        delta, self.pending = self.pending, None
+        post, self.pending_post = self.pending_post, None
+        if delta is not None and post is None:
+            raise RuntimeError("the stream holds a delta that is added without a norm; a norm has to read it first")
+        if rt.dtype == torch.float32 and delta is None:
+            return self.x
+        out = None if rt.dtype == torch.float32 else torch.empty(self.x.shape, dtype=rt.dtype, device=self.x.device)
+        rt.ops.add_normed(self.x, delta, post, out, rt.dtype)
+        return self.x if out is None else out
 
     def add(self, delta, post=None) -> None:
         """``post`` = (weight, eps, mult): the delta is normed and scaled before it is added (see ``Norm``)."""

@@ -88,6 +88,27 @@ class SandwichBlock(PreNormBlock):
         stream.add(self.ffn.forward(h, ctx), post=(self.post2.weighted(), s.post2.eps, s.residual_mult))
 
 
+@register_part("block", "outnorm")
+class OutNormBlock(PreNormBlock):
+    """x += norm1(mixer(x)); x += norm2(ffn(x)): a sublayer reads the stream as it is, and its result is normed (root mean
+    square, weight) before the residual sum.  One kernel a sublayer norms the pending result in 32-bit, adds it and leaves the
+    sum in the compute dtype for the sublayer that reads it next."""
+
+    def __init__(self, spec, prefix, rt):
+        super().__init__(spec, prefix, rt)
+        for n in (spec.norm1, spec.norm2):
+            if n is not None and (n.kind != "rmsnorm" or n.groups != 1):
+                raise ValueError("outnorm block: the norm of a sublayer's result is a root-mean-square norm over the whole row")
+
+    def forward(self, stream, ctx, cache):
+        h = stream.plain(self.rt)
+        stream.add(self.mixer.forward(h, ctx, cache), post=(self.norm1.weighted(), self.spec.norm1.eps, 1.0))
+        if self.ffn is None:
+            return
+        h = stream.plain(self.rt)
+        stream.add(self.ffn.forward(h, ctx), post=(self.norm2.weighted(), self.spec.norm2.eps, 1.0))
+
+
 def _register_stream_initialisers():
     """Starts of the random-weights mode under which several streams keep the size of one: a sublayer reads about the mean
     of the streams, writes about as much as it returns into each, and the streams stay mostly themselves."""

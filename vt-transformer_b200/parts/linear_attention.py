@@ -1,6 +1,6 @@
 """Mixers that carry a matrix of fixed size for each request and head instead of keys and values: gated linear
-attention, the generalized delta rule, the delta rule with one decay a head and the matrix memory with exponential
-gates.  The state lives in 32-bit in a ``StateSpec`` slot of the cache manager
+attention, the generalized delta rule, the delta rule with one decay a head, the matrix memory with exponential
+gates and the state-space recurrence.  The state lives in 32-bit in a ``StateSpec`` slot of the cache manager
 (zero when a request is admitted), and one kernel walks a step's tokens of every (request, head) in order, a single
 decoded token and a portion of a prompt alike."""
 from __future__ import annotations
@@ -337,3 +337,77 @@ class MatrixMemory(_Recurrent):
                         s.den_eps, cache.state, ctx, o, s.heads, s.dim, s.v_dim, status=ctx.status)
         ops.head_norm_gate(o, y, cols[3], self.norm, True, s.norm_eps, "sigmoid", out, out_col, out_scale, s.heads, s.v_dim,
                            token_seq=ctx.token_seq)
+
+
+def _log_rates(shape, g, sigma, device):
+    """Logarithms of decay rates in the random-weights mode: rates from about 1/8 to 8, so that some heads forget at once and
+    others keep what they have for many tokens."""
+    return (torch.rand(shape, generator=g, dtype=torch.float32, device=device) - 0.5) * 4.0
+
+
+def _register_log_rates():
+    from ..weights.loader import register_initialiser
+    register_initialiser("log_rates", _log_rates, replace=True)
+
+
+_register_log_rates()
+
+
+@register_part("mixer", "state_space")
+class StateSpace(_Recurrent):
+    """See ``StateSpaceSpec``.  z, the convolution's inputs and dt are one product (the rows of the stored matrix cut in three,
+    each starting at a multiple of 8 columns); one kernel runs the convolution with its bias and silu and renews the kept
+    inputs; the scan forms step sizes and decays in 32-bit and walks the tokens (or, for portions in bfloat16, works chunk by
+    chunk, see ``ops.state_space``); one kernel gates the result, norms its groups and multiplies by the weight."""
+
+    def __init__(self, spec, prefix, rt):
+        super().__init__(spec, prefix, rt)
+        if spec.heads % spec.groups:
+            raise ValueError(f"state space: {spec.heads} heads over {spec.groups} groups")
+        self.inner = spec.heads * spec.v_dim
+        if self.inner % spec.norm_groups:
+            raise ValueError(f"state space: {self.inner} values in {spec.norm_groups} norm groups")
+        if not 1 <= spec.taps <= 16:
+            raise ValueError(f"state space: a convolution of {spec.taps} taps; 1 to 16 are built")
+        self.channels = self.inner + 2 * spec.groups * spec.dim
+
+    def cache_spec(self):
+        s = self.spec
+        state = StateSpec((s.heads, s.dim, s.v_dim), torch.float32)
+        if s.taps == 1:
+            return state
+        return (state, StateSpec((s.taps - 1, self.channels), torch.float32))
+
+    def param_specs(self):
+        s, p = self.spec, self.prefix
+        w_in, conv, conv_b, dt, a_log, d, norm, o = s.names
+        return {p + w_in: ParamSpec((self.inner + self.channels + s.heads, s.hidden)), p + o: ParamSpec((s.hidden, self.inner)),
+                p + conv: ParamSpec((self.channels, s.taps), role="vector", init="conv_taps"),
+                p + conv_b: ParamSpec((self.channels,), role="vector"), p + dt: ParamSpec((s.heads,), role="vector"),
+                p + a_log: ParamSpec((s.heads,), role="vector", init="log_rates"),
+                p + d: ParamSpec((s.heads,), role="vector", init="one_plus_normal"),
+                p + norm: ParamSpec((self.inner,), role="vector", init="one_plus_normal")}
+
+    def load(self, get) -> None:
+        s, p, rt = self.spec, self.prefix, self.rt
+        w_in, conv, conv_b, dt, a_log, d, norm, o = s.names
+        self._in = list(torch.split(rt.param(get(p + w_in)), [self.inner, self.channels, s.heads]))
+        self.w_o = rt.param(get(p + o))
+        self.conv = rt.param(get(p + conv), "vector").t().contiguous()         # [taps, channels]: a tap's weights side by side
+        self.conv_bias, self.dt_bias, self.a_log, self.d, self.norm = (rt.param(get(p + n), "vector") for n in (conv_b, dt, a_log, d, norm))
+        self._small = (self.conv, self.conv_bias, self.dt_bias, self.a_log, self.d, self.norm)
+        self.pack()
+
+    def inner_size(self) -> int:
+        return self.inner
+
+    def core(self, y, cols, ctx, cache, out, out_col, out_scale) -> None:
+        s, ops = self.spec, self.rt.ops
+        state, tail = (cache[0].state, cache[1].state) if isinstance(cache, (tuple, list)) else (cache.state, None)
+        u = torch.empty((y.shape[0], self.channels), dtype=y.dtype, device=y.device)
+        ops.causal_conv(y, cols[1], self.conv, self.conv_bias, tail, ctx, u, silu=True, status=ctx.status)
+        o = torch.empty((y.shape[0], self.inner), dtype=torch.float32, device=y.device)
+        ops.state_space(u, y, cols[2], self.a_log, self.dt_bias, self.d, state, ctx, o, s.heads, s.groups, s.dim, s.v_dim, status=ctx.status)
+        # the norm's groups are heads as wide as a group, with a weight for every channel and the gate in front
+        ops.head_norm_gate(o, y, cols[0], self.norm, True, s.norm_eps, "silu", out, out_col, out_scale, s.norm_groups,
+                           self.inner // s.norm_groups, token_seq=ctx.token_seq, gate_first=True)

@@ -200,6 +200,8 @@ class Experts(FeedForward):
                 out[prefix + g] = ParamSpec((inter, s.hidden))
             out[prefix + u] = ParamSpec((inter, s.hidden))
             out[prefix + d] = ParamSpec((s.hidden, inter))
+        if s.router_bias_name is not None:
+            out[p + s.router_bias_name] = ParamSpec((s.experts,), role="vector")
         if s.shared_gate_name is not None:
             out[p + s.shared_gate_name] = ParamSpec((1, s.hidden))
         return out
@@ -208,6 +210,7 @@ class Experts(FeedForward):
         s, p, rt = self.spec, self.prefix, self.rt
         g, u, d = s.names
         self.router = rt.param(get(p + s.router_name), "vector")       # [experts, hidden] in 32-bit
+        self.router_bias = rt.param(get(p + s.router_bias_name), "vector") if s.router_bias_name is not None else None
         self.inter = -(-s.inter // 8) * 8
         blocks = [(f"{p}{s.expert_prefix}{e}.", s.inter, self.inter) for e in range(s.experts)]
         if s.shared_inter:
@@ -238,7 +241,7 @@ class Experts(FeedForward):
         self.down_of = [d.contiguous() for d in down]
 
     def weight_bytes(self) -> int:
-        mats = (self.router, self.w_gate_up, self.w_down, self.shared_gate)
+        mats = (self.router, self.w_gate_up, self.w_down, self.shared_gate, self.router_bias)
         return sum(m.numel() * m.element_size() for m in mats if m is not None)
 
     def first_product(self):
@@ -254,7 +257,7 @@ class Experts(FeedForward):
                      split=s.experts * self.inter, limit2=s.shared_limit if s.shared_inter else None)
         # the router's logits are formed there, in 32-bit (and the shared expert's gate)
         ops.route_experts(None, s.top, act, self.inter, x=h, router=self.router, weights_by=s.router_weights, scale=s.router_scale,
-                          shared_gate=self.shared_gate)
+                          shared_gate=self.shared_gate, bias=self.router_bias)
         return ops.linear_to_stream(act, self.w_down, None, then=self.then)
 
     def grouped(self, h):
@@ -265,7 +268,7 @@ class Experts(FeedForward):
         weights = torch.empty((T, s.top), dtype=torch.float32, device=dev)
         gates = None if self.shared_gate is None else torch.empty((T,), dtype=torch.float32, device=dev)
         ops.route_topk(None, s.top, ids, weights, x=h, router=self.router, weights_by=s.router_weights, scale=s.router_scale,
-                       shared_gate=self.shared_gate, gates=gates)
+                       shared_gate=self.shared_gate, gates=gates, bias=self.router_bias)
         lists = torch.empty((s.experts, T), dtype=torch.int32, device=dev)
         counts = torch.empty((s.experts,), dtype=torch.int32, device=dev)
         ops.expert_lists(ids, lists, counts)

@@ -46,13 +46,14 @@ class NoPosition(PositionEncoding):
         self.table = None
 
 
-def rotation_frequencies(dim: int, base: float, scaling=None) -> torch.Tensor:
+def rotation_frequencies(dim: int, base: float, scaling=None, divide_by: float = 1.0) -> torch.Tensor:
     """[dim / 2] float32: base^(-2i/dim), formed in double and rounded once.  ``scaling`` = (factor, low, high,
     original): a frequency f with wavelength l = 2 pi / f stays where l < original / high, becomes f / factor where
-    l > original / low, and between the two (1 - s) f / factor + s f with s = (original / l - low) / (high - low)."""
+    l > original / low, and between the two (1 - s) f / factor + s f with s = (original / l - low) / (high - low).  ``divide_by``: every
+    frequency is divided by it."""
     out = []
     for i in range(dim // 2):
-        f = math.pow(float(base), -2.0 * i / dim)
+        f = math.pow(float(base), -2.0 * i / dim) / divide_by
         if scaling is not None:
             factor, low, high, original = (float(v) for v in scaling)
             wavelength = 2.0 * math.pi / f
@@ -79,13 +80,15 @@ class ComputedRotary(PositionEncoding):
         self.frequencies, self.mult = None, 1.0
         if not self.spec.dim:
             return
+        if self.spec.scaling is not None and self.spec.factor != 1.0:
+            raise ValueError("rotary_computed: one of 'scaling', 'ramp' and 'factor'")
         if self.spec.ramp is not None:
-            if self.spec.scaling is not None:
-                raise ValueError("rotary_computed: either 'scaling' or 'ramp'")
+            if self.spec.scaling is not None or self.spec.factor != 1.0:
+                raise ValueError("rotary_computed: one of 'scaling', 'ramp' and 'factor'")
             f, self.mult = ramped_frequencies(self.spec.dim, self.spec.base, self.spec.ramp)
             self.frequencies = f.to(self.rt.device)
         else:
-            self.frequencies = rotation_frequencies(self.spec.dim, self.spec.base, self.spec.scaling).to(self.rt.device)
+            self.frequencies = rotation_frequencies(self.spec.dim, self.spec.base, self.spec.scaling, self.spec.factor).to(self.rt.device)
 
 
 def ramped_frequencies(dim: int, base: float, ramp=None):

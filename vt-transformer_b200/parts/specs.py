@@ -44,13 +44,15 @@ class PositionSpec:
     ``rotary_interleaved``: pairs (2i, 2i + 1) of the first ``dim`` dimensions, angle formed where it is used as for
     ``rotary_computed``.  ``ramp`` (``rotary_interleaved`` and ``rotary_computed``) = (factor, original, fast, slow): with n(t) = dim ln(original / (2 pi t)) / (2 ln base),
     lo = max(floor(n(fast)), 0), hi = min(ceil(n(slow)), dim - 1) and r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1),
-    pair i turns with f_i / factor * r_i + f_i (1 - r_i), and cos and sin are multiplied by 0.1 ln(factor) + 1."""
+    pair i turns with f_i / factor * r_i + f_i (1 - r_i), and cos and sin are multiplied by 0.1 ln(factor) + 1.
+    ``factor`` (``rotary_computed`` without the two above): every frequency is divided by it."""
     dim: int = 0
     base: float = 0.0
     max_positions: int = 0
     kind: str = "rotary"
     scaling: Optional[Tuple[float, float, float, float]] = None
     ramp: Optional[Tuple[float, float, float, float]] = None
+    factor: float = 1.0
 
 
 @dataclass(frozen=True)
@@ -85,6 +87,10 @@ class AttentionSpec(MixerSpec):
     # projection and multiplied by a weight of that size (``norm_names`` below the part's prefix)
     proj_norm_eps: Optional[float] = None
     norm_names: Tuple[str, str] = ("q.norm", "k.norm")
+    # e: before the rotation every head of q and of k is divided by its own sqrt(mean(.^2) + e) and multiplied by a weight
+    # [head_dim] (``norm_names``), one for q and one for k, shared by the heads
+    head_norm_eps: Optional[float] = None
+    values_from_keys: bool = False         # there is no v projection: a value is its key's projection, before norm and rotation
     q_temp: Optional[Tuple[float, int]] = None   # (c, n): q at position p is multiplied by 1 + c ln(floor((p + 1) / n) + 1)
     softcap: Optional[float] = None        # c: score <- c tanh(score / c) after the scale
     # "zero": the softmax's denominator holds one more term exp(0); "learned": exp(s_h), s [heads] the tensor ``sink_name``;
@@ -149,7 +155,9 @@ class LatentAttentionSpec(MixerSpec):
     U_v,i c (``v_dim``); score = q . k * ``scale``; causal softmax, with ``sink`` one more term exp(s_i) (a number a head) in
     the denominator; ``gate`` "element": the heads' results are multiplied element by element by sigmoid(G h), "head": head
     i's by sigmoid(G h)_i (G [heads, hidden]); then the output projection.  ``window`` None sees all earlier tokens; w sees
-    token j from position p if p - w < j <= p.
+    token j from position p if p - w < j <= p.  ``own_latent`` False: the layer has no D_kv (and no norm of it); c and the shared
+    key part are those that the run which wrote its cache slot has stored (``RunSpec.writes`` False), read with this layer's own
+    U_k, U_v, queries and window.
     ``names``: D_q, its norm, U_q, D_kv, its norm, U_k, U_v, output, sink, gate."""
     hidden: int = 0
     heads: int = 0
@@ -162,6 +170,7 @@ class LatentAttentionSpec(MixerSpec):
     sink: bool = False
     gate: str = "none"
     window: Optional[int] = None
+    own_latent: bool = True
     norm_eps: float = 1e-6
     position: PositionSpec = field(default_factory=lambda: PositionSpec(kind="none"))
     names: Tuple[str, ...] = ("dq", "dq.norm", "uq", "dkv", "dkv.norm", "uk", "uv", "o", "sink", "g")
@@ -268,6 +277,28 @@ class MatrixMemorySpec(MixerSpec):
 
 
 @dataclass(frozen=True)
+class StateSpaceSpec(MixerSpec):
+    """A state-space recurrence with one decay a token and head.  in h = [z | x | B | C | dt] with z and x of ``heads`` *
+    ``v_dim``, B and C of ``groups`` * ``dim`` and dt of ``heads`` rows.  x, B and C together pass a causal convolution over time,
+    channel by channel (``taps`` taps, the last one the present token's, zeros before a request's first token; tensor [channels,
+    taps] and bias [channels]) and silu.  With d = softplus(dt[h] + dt_bias[h]) and S [dim, v_dim] a head (32-bit, zero at the
+    start of a request; head h with group h // (heads / groups)): S <- exp(-exp(A_log[h]) d) S + d B x^T, y = S^T C + D[h] x.  The
+    heads' y together are multiplied by silu(z), cut into ``norm_groups`` equal parts, each divided by its own root mean square
+    (``norm_eps``), and multiplied by a weight [heads * v_dim]; then the output projection.  A request keeps S and the last
+    taps - 1 inputs of the convolution.  ``names``: in, convolution, its bias, dt_bias, A_log, D, the norm's weight, output."""
+    hidden: int = 0
+    heads: int = 0
+    groups: int = 1
+    dim: int = 0
+    v_dim: int = 0
+    taps: int = 1
+    norm_groups: int = 1
+    norm_eps: float = 1e-6
+    names: Tuple[str, ...] = ("in", "conv", "conv.b", "dt_bias", "A_log", "D", "norm", "o")
+    kind: str = "state_space"
+
+
+@dataclass(frozen=True)
 class NormedParallelSpec(MixerSpec):
     """Several mixers side by side on the same input, each result normed before the sum:
     sum_i scales[i] * w_i * y_i / sqrt(mean(y_i^2) + eps) with y_i = branches[i](h) after its own output projection and w_i
@@ -345,7 +376,7 @@ class ExpertsSpec(FeedForwardSpec):
     it, times ``router_scale``).
     ``activation`` "relu_square": the experts have no gate matrix, an expert is down(max(up(x), 0)^2).  ``shared_gate_name``: the
     shared expert's result is multiplied by sigmoid(g . x), g [1, hidden] the tensor of that name below the part's prefix
-    (32-bit)."""
+    (32-bit).  ``router_bias_name``: z = R x + b with b [experts] the tensor of that name below the part's prefix."""
     hidden: int = 0
     experts: int = 0
     top: int = 1
@@ -362,6 +393,7 @@ class ExpertsSpec(FeedForwardSpec):
     expert_prefix: str = "e"
     shared_prefix: str = "shared."
     shared_gate_name: Optional[str] = None
+    router_bias_name: Optional[str] = None
     kind: str = "experts"
 
 
@@ -374,6 +406,8 @@ class BlockSpec:
     after the sums and their result is the stream.  With ``shift_name`` the mixer reads h_t + (h_(t-1) - h_t) * mu
     (mu [hidden] the tensor of that name below the layer's prefix, h_(t-1) the previous token's x, zeros before a request's
     first token), and the layer keeps a request's last x beside what its mixer keeps.
+
+    ``outnorm``: x += norm1(mixer(x)); x += norm2(ffn(x)): the norms are of the sublayers' results, which read x as it is.
 
     ``streams`` (the model's residual is several streams x_s): sublayer q = 1, 2 reads u = sum_s in[s] x_s and all streams
     change at once, x_t <- sum_s mix[s, t] x_s + out[t] sublayer(h), h = norm(u); in, out [streams] and mix [streams, streams]
@@ -413,7 +447,7 @@ class RunSpec:
 
     Cache slots are numbered by the model; a slot belongs to the run that writes it.  A
     run with ``writes=False`` reads a slot that an earlier run wrote (shared keys and
-    values) and stores nothing.  A block may appear in several runs, each with a slot of
+    values) and stores nothing; a slot that several runs read keeps what the widest of their windows sees.  A block may appear in several runs, each with a slot of
     its own.  For a block whose mixer keeps several things (``Mixer.cache_spec`` returns a tuple) ``cache`` is a tuple
     of slots, one for each, in that order.  ``add_embedding``: before this run the embedding's output (the stream as it
     was before the first run) is added to the stream once more."""
