@@ -461,6 +461,28 @@ def _laposun_config(width, ff, att, window, layers=4):
                        for i in range(layers)]}
 
 
+def _gedulorn_config(width, ff, att, window):
+    """An attention layer (values that are the keys' projections, normed queries and keys, half of each head rotated, capped
+    scores) and two latent-attention layers with sinks, the second over the first one's latent, all under a window, and after
+    the attention a state-space layer (heads of 64 with 2 ``width`` values together, a state of 128, a group for every 16 heads,
+    4 taps); every layer with 8 experts of which a token uses 2 beside a shared expert, the three experts a token runs having
+    ``ff`` inner values together.  ``att``: (heads, kv heads, head size) of the Qwen2 model of equal size; the latents as for Geponex."""
+    heads, kv_heads, dim = att
+    inner, n = ff // 3 // 64 * 64, 2 * width // 64
+    moe = {"kind": "moe", "router": {"experts": 8, "top": 2}, "expert": {"ff": inner}, "shared": {"ff": inner}}
+    mask = {"size": window}
+    latent = {"heads": heads, "dim": dim, "rot_dim": dim // 2, "vdim": dim, "q_rank": 12 * dim, "kv_rank": 4 * dim, "scale": (1.5 * dim) ** -0.5,
+              "rot": {"dims": dim // 2, "base": 1e6}, "mask": mask}
+    layers = [
+        {"type": "attention", "mlp": moe, "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "softcap": 50.0,
+                                                    "rot": {"dims": dim // 2, "base": 1e6, "scaling": {"factor": 4.0}}, "mask": mask}},
+        {"type": "mamba2", "mlp": moe, "mixer": {"heads": n, "vdim": 64, "state": 128, "groups": n // 16, "conv": 4, "norm_groups": n // 16}},
+        {"type": "latent_attention", "mlp": moe, "mixer": latent},
+        {"type": "latent_attention", "mlp": moe, "mixer": dict(latent, kv_from=2)},
+    ]
+    return {"architecture": "Gedulorn", "vocab": 32768, "width": width, "embedding": {"scale": 32.0}, "norm": {"eps": 1e-6}, "layers": layers}
+
+
 DESIGN_SIZES = {
     # name: width, feed-forward, (gla heads, dim, vdim), (attention heads, kv heads, head size), (delta heads, dim), chunk
     "w1024": (1024, 4096, (8, 64, 128), (16, 2, 64), (8, 64), 1024),
@@ -476,9 +498,11 @@ DESIGNS = {
     "fosepel": lambda width, ff, gla, att, delta, chunk: _fosepel_config(width, ff, gla, att, delta),
     # (the window is the other design's chunk)
     "laposun": lambda width, ff, gla, att, delta, chunk: _laposun_config(width, ff, att, chunk),
+    "gedulorn": lambda width, ff, gla, att, delta, chunk: _gedulorn_config(width, ff, att, chunk),
 }
-# a design whose mixers and experts are another design's with other options is measured beside that one too
-CLOSEST = {"laposun": "geponex"}
+# a design whose mixers and experts are other designs' with other options is measured beside those too (the last one's latent
+# attention is the second, its capped attention and recurrences are the first)
+CLOSEST = {"laposun": ("geponex",), "gedulorn": ("fosepel", "laposun")}
 
 
 def design_points(design: str, sizes, steps: int, warmup: int) -> int:
@@ -513,7 +537,7 @@ def design_points(design: str, sizes, steps: int, warmup: int) -> int:
 
     def per_kernel(runner, entries):
         """Device time of each of the package's kernels in one eager step, by the name of the op."""
-        names = [n for n in ("embedding", "rmsnorm", "layernorm", "polynorm", "head_norm_gate", "gla_scan", "delta_scan",
+        names = [n for n in ("add_normed", "causal_conv", "state_space", "embedding", "rmsnorm", "layernorm", "polynorm", "head_norm_gate", "gla_scan", "delta_scan",
                              "retention_scan", "gated_delta_scan", "conv_tail_update", "memory_scan", "embedding_pair", "streams_norm", "relu_square", "linear_relu_square", "expert_lists", "gather_picks", "combine_picks", "normed_sum", "add_rows", "route_experts", "route_topk", "token_shift", "latent_prepare", "head_matmul", "attention_latent", "xielu",
                              "gate_clamp", "attention_differential", "attention_prepare", "attention_general", "rope_store", "paged_attention", "rope_attention", "linear",
                              "linear_silu_mul", "linear_to_stream", "logits_scale_cap") if hasattr(ops, n)]
@@ -555,8 +579,8 @@ def design_points(design: str, sizes, steps: int, warmup: int) -> int:
                           num_hidden_layers=4, num_attention_heads=att[0], num_key_value_heads=att[1], head_dim=att[2],
                           rms_norm_eps=1e-6, rope_theta=1e6, max_position_embeddings=8192, tie_word_embeddings=True),
         }
-        if design in CLOSEST:
-            models[CLOSEST[design]] = DESIGNS[CLOSEST[design]](width, ff, gla, att, delta, chunk)
+        for close in CLOSEST.get(design, ()):
+            models[close] = DESIGNS[close](width, ff, gla, att, delta, chunk)
         res = {}
         for name, raw in models.items():
             cfg = config_from_dict(raw)

@@ -124,6 +124,9 @@ def plain_module(folder: str):
     if c.get("architecture") == "Laposun":
         from plain import laposun_plain
         return laposun_plain
+    if c.get("architecture") == "Gedulorn":
+        from plain import gedulorn_plain
+        return gedulorn_plain
     if c.get("architecture") == "Fosepel":
         from plain import fosepel_plain
         return fosepel_plain
