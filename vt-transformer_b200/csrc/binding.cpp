@@ -706,6 +706,24 @@ struct RouterInput {
     int width = 0, tokens = 0, experts = 0, x_dtype = vtb::kF32;
 };
 
+void state_space_chunks(const Tensor& u, const Tensor& y, int64_t dt_col, const Tensor& a_log, const Tensor& dt_bias, const Tensor& d, Tensor& state,
+                        const Tensor& cu_q, const Tensor& rows, const Tensor& walks, const Tensor& chunks, Tensor& starts, Tensor& o, int64_t heads,
+                        int64_t groups, int64_t dim, int64_t v_dim, c10::optional<Tensor> status) {
+    check_space(u, y, dt_col, a_log, dt_bias, d, state, cu_q, rows, o, heads, groups, dim, v_dim, "state_space_chunks");
+    TORCH_CHECK(y.scalar_type() == torch::kBFloat16, "state_space_chunks: bfloat16 only");
+    TORCH_CHECK(vtb::state_space_chunks_supports(heads, groups, dim, v_dim) && u.size(1) % 8 == 0,
+                "state_space_chunks: a state size that is a multiple of 8 up to 256, values a multiple of 8");
+    check_i32(walks, "walks"); check_i32(chunks, "chunks"); check_f32(starts, "starts");
+    TORCH_CHECK(walks.dim() == 2 && walks.size(1) == 2 && chunks.dim() == 2 && chunks.size(1) == 2, "state_space_chunks: walks and chunks [n, 2]");
+    TORCH_CHECK(starts.numel() >= chunks.size(0) * heads * dim * v_dim, "state_space_chunks: a state for every chunk");
+    c10::cuda::CUDAGuard guard(y.device());
+    check_launch(vtb::launch_state_space_chunks(u.data_ptr(), u.size(1), y.data_ptr(), y.size(1), dt_col, a_log.data_ptr<float>(),
+                                                dt_bias.data_ptr<float>(), d.data_ptr<float>(), state.data_ptr<float>(), state.size(0),
+                                                cu_q.data_ptr<int>(), rows.data_ptr<int>(), rows.numel(), walks.data_ptr<int>(), walks.size(0),
+                                                chunks.data_ptr<int>(), chunks.size(0), starts.data_ptr<float>(), o.data_ptr<float>(), heads,
+                                                groups, dim, v_dim, status_ptr(status), stream_of(y)), "state_space_chunks");
+}
+
 // a number for every expert that is added to its logit
 const float* router_bias(const c10::optional<Tensor>& bias, int experts, const char* who) {
     if (!bias.has_value()) return nullptr;
@@ -1484,6 +1502,10 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
     m.def("state_space_scan", &state_space_scan, py::arg("u"), py::arg("y"), py::arg("dt_col"), py::arg("a_log"), py::arg("dt_bias"), py::arg("d"),
           py::arg("state"), py::arg("cu_q"), py::arg("rows"), py::arg("seqs"), py::arg("o"), py::arg("heads"), py::arg("groups"), py::arg("dim"),
           py::arg("v_dim"), py::arg("status") = py::none());
+    m.def("state_space_chunks", &state_space_chunks, py::arg("u"), py::arg("y"), py::arg("dt_col"), py::arg("a_log"), py::arg("dt_bias"), py::arg("d"),
+          py::arg("state"), py::arg("cu_q"), py::arg("rows"), py::arg("walks"), py::arg("chunks"), py::arg("starts"), py::arg("o"), py::arg("heads"),
+          py::arg("groups"), py::arg("dim"), py::arg("v_dim"), py::arg("status") = py::none());
+    m.def("state_space_chunks_supports", &vtb::state_space_chunks_supports);
     m.def("gla_scan", &gla_scan, py::arg("y"), py::arg("q_col"), py::arg("k_col"), py::arg("v_col"), py::arg("low_col"), py::arg("a2"),
           py::arg("a2_bias"), py::arg("inv_tau"), py::arg("q_scale"), py::arg("state"), py::arg("cu_q"), py::arg("rows"), py::arg("o"),
           py::arg("heads"), py::arg("dim"), py::arg("v_dim"), py::arg("status") = py::none(), py::arg("most_threads") = 0);

@@ -43,6 +43,7 @@ SOURCES = [
     "latent.cu",
     "streams.cu",
     "state_space.cu",
+    "state_space_chunks.cu",
 ]
 HEADERS = ["common.cuh", "kernels.h", "launch.cuh", "tc_common.cuh", "gemm_epilogue.cuh", "attention_mma.cuh", "attention_decode.cuh", "attention_noalloc.h", "look_ahead.cuh"]
 

@@ -80,6 +80,15 @@ cudaError_t launch_state_space_scan(int dtype, const void* u, int u_stride, cons
                                     int n_seqs, const int* seqs, int n_listed, float* out, int heads, int groups, int dim, int v_dim, int* status,
                                     cudaStream_t stream);
 
+// The same recurrence over portions in bfloat16, chunk by chunk of 64 tokens on the tensor cores (state_space_chunks.cu): walks [n_walks, 2]
+// (sequence, its first chunk), chunks [n_chunks, 2] (sequence, first of its new tokens), a sequence's chunks one after the other;
+// starts [n_chunks, heads, dim, v_dim] scratch.  dim a multiple of 8 up to 256, v_dim a multiple of 8.
+bool state_space_chunks_supports(int heads, int groups, int dim, int v_dim);
+cudaError_t launch_state_space_chunks(const void* u, int u_stride, const void* y, int stride, int dt_col, const float* a_log, const float* dt_bias,
+                                      const float* d, float* state, int state_rows, const int* cu_q, const int* rows, int n_seqs,
+                                      const int* walks, int n_walks, const int* chunks, int n_chunks, float* starts, float* out, int heads,
+                                      int groups, int dim, int v_dim, int* status, cudaStream_t stream);
+
 // Recurrences with one decay a head (recurrent_gated.cu), in the manner of the scans above: q, k, v and the gates' inputs are
 // columns of y; the state is read at rows[sequence] and left as after the sequence's last token; out [tokens, heads * v_dim].
 // The delta rule with one decay a head: q and k [kv_heads * dim], v [heads * v_dim] pass a causal convolution over time

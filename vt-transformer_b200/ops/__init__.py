@@ -302,15 +302,64 @@ def causal_conv(y, col: int, w: torch.Tensor, bias, tail, ctx, out: torch.Tensor
     return out
 
 
+STATE_SPACE_CHUNK = 64           # tokens of a chunk of the tensor-core kernels
+# A sequence that brings this many tokens in a bfloat16 step goes through those kernels; a shorter one (a single token beside
+# portions of prompts) is walked token by token.
+STATE_SPACE_CHUNK_MIN = int(os.environ.get("VTB200_STATE_SPACE_CHUNK_MIN", "16"))
+
+
+class _ChunkPlan:
+    """How a step's sequences go through the state-space kernels: ``short`` (int32 indices, or None) token by token, the others
+    chunk by chunk: ``walks`` (sequence, its first chunk), ``chunks`` (sequence, first of its new tokens)."""
+
+    def __init__(self, ctx, device):
+        short, walks, chunks = [], [], []
+        for i, s in enumerate(ctx.seqs):
+            if s.length < STATE_SPACE_CHUNK_MIN:
+                short.append(i)
+                continue
+            walks.append((i, len(chunks)))
+            chunks += [(i, t) for t in range(0, s.length, STATE_SPACE_CHUNK)]
+        self.n_chunks = len(chunks)
+        if not chunks:
+            return
+        flat = [v for pair in walks + chunks for v in pair] + short
+        host = torch.tensor(flat, dtype=torch.int32)
+        if torch.device(device).type == "cuda":
+            host = host.pin_memory()
+        buf, a, b = host.to(device, non_blocking=True), 2 * len(walks), 2 * (len(walks) + len(chunks))
+        self.walks, self.chunks = buf[:a].view(-1, 2), buf[a:b].view(-1, 2)
+        self.short = buf[b:] if short else None
+
+
 def state_space(u, y, dt_col: int, a_log, dt_bias, d, state: torch.Tensor, ctx, o: torch.Tensor, heads: int, groups: int, dim: int,
                 v_dim: int, status=None) -> torch.Tensor:
     """A state-space recurrence over the step's tokens, sequence by sequence and head by head.  ``u`` [T, heads * v_dim +
     2 groups * dim] holds x, B and C side by side; the raw step size of head h is y[t, dt_col + h].  With s = softplus(raw + dt_bias[h]):
     S <- exp(-exp(a_log[h]) s) S + s B x^T, o = S^T C + d[h] x, head h with group h // (heads / groups).  ``state`` [request rows,
     heads, dim, v_dim] float32 is read at the step's ``ctx.rows`` and left as after the last token; ``o`` [T, heads * v_dim] float32.
-    Step sizes, decays, state and sums in 32-bit."""
-    backend().state_space_scan(u, y, int(dt_col), a_log, dt_bias, d, state, ctx.cu_q, ctx.rows, None, o, int(heads), int(groups), int(dim),
-                               int(v_dim), status)
+    Step sizes, decays, state and sums in 32-bit.
+
+    Portions in bfloat16 at the sizes the tensor-core kernels take go chunk by chunk: one kernel walks a sequence's chunks and
+    leaves the state before each, one forms all chunks' outputs side by side.  Everything else goes token by token."""
+    global launches
+    be = backend()
+    sizes = (int(heads), int(groups), int(dim), int(v_dim))
+    short = None
+    if ctx.max_q_len >= STATE_SPACE_CHUNK_MIN and ctx.seqs and y.dtype == torch.bfloat16 and be.state_space_chunks_supports(*sizes):
+        key = ("state_space_plan", STATE_SPACE_CHUNK_MIN)
+        plan = ctx.extras.get(key)
+        if plan is None:
+            plan = ctx.extras[key] = _ChunkPlan(ctx, y.device)
+        if plan.n_chunks:
+            starts = torch.empty((plan.n_chunks, heads, dim, v_dim), dtype=torch.float32, device=y.device)
+            launches += 1
+            be.state_space_chunks(u, y, int(dt_col), a_log, dt_bias, d, state, ctx.cu_q, ctx.rows, plan.walks, plan.chunks, starts, o, *sizes, status)
+            if plan.short is None:
+                return o
+            launches += 1
+            short = plan.short
+    be.state_space_scan(u, y, int(dt_col), a_log, dt_bias, d, state, ctx.cu_q, ctx.rows, short, o, *sizes, status)
     return o
 
 
