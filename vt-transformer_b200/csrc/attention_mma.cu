@@ -102,7 +102,7 @@ attention_mma_kernel(const AttnParams p) {
             lrow[i] = tq == 0 ? 1.f : 0.f;
         }
     }
-    const float cap = p.softcap, cap_log2 = p.softcap * 1.4426950408889634f, over_cap = p.softcap > 0.f ? p.scale / p.softcap : 0.f;
+    const float cap = p.softcap, cap_log2 = p.softcap * 1.4426950408889634f, over_cap = p.softcap > 0.f ? p.scale / p.softcap * 2.8853900817779268f : 0.f;
 
     const int* table = p.block_table + (size_t)seq * p.table_stride;
     auto load_block = [&](int blk, int stage) {
@@ -179,7 +179,7 @@ attention_mma_kernel(const AttnParams p) {
             for (int j = 0; j < KB / 8; ++j) {
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
-                    s[j][e] = cap > 0.f ? cap_log2 * tanhf(s[j][e] * over_cap) : s[j][e] * p.scale_log2;
+                    s[j][e] = cap > 0.f ? cap_log2 * cap_tanh(s[j][e] * over_cap) : s[j][e] * p.scale_log2;
                     mnew[e >> 1] = fmaxf(mnew[e >> 1], s[j][e]);
                 }
             }
@@ -191,7 +191,7 @@ attention_mma_kernel(const AttnParams p) {
                     const int i = e >> 1;
                     const int key = kb + j * 8 + 2 * tq + (e & 1);
                     const bool see = valid[i] && key <= pos[i] && key >= first_visible_key(pos[i], p.window, p.chunk);
-                    s[j][e] = see ? (cap > 0.f ? cap_log2 * tanhf(s[j][e] * over_cap) : s[j][e] * p.scale_log2) : -INFINITY;
+                    s[j][e] = see ? (cap > 0.f ? cap_log2 * cap_tanh(s[j][e] * over_cap) : s[j][e] * p.scale_log2) : -INFINITY;
                     mnew[i] = fmaxf(mnew[i], s[j][e]);
                 }
             }

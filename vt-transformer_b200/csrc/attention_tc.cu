@@ -54,7 +54,8 @@ struct AttnTcParams {
     int table_stride;
     const int2* tiles;
     int n_pages, heads, kv_heads, page_size, window, chunk;
-    float scale_log2;
+    float scale_log2;        // scale * log2(e), or the cap * log2(e) where scores are capped
+    float over_cap;          // 2 log2(e) * scale / cap
     int tokens_per_tile;
     int run_keys;            // keys of a run: 16, 32, 64 or 128, a divisor of the page size
     int cache_rows;          // pages * kv_heads * page_size: a row index beyond it makes TMA fill zeros
@@ -140,7 +141,7 @@ __device__ __forceinline__ void write_p_half(const uint32_t (&raw)[TK], uint32_t
     }
 }
 
-template <int D>
+template <int D, bool CAP>
 __global__ void __launch_bounds__(ATC_THREADS)
 attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                     const AttnTcParams p) {
@@ -337,6 +338,11 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
             const bool open = (kb + TK - 1 <= pos_lo) && kb >= first_visible_key(pos_hi, p.window, p.chunk);
             uint32_t raw[TK];
             load_row(s_addr, raw);
+            if constexpr (CAP) {
+                // score = cap * tanh(scale * raw / cap): the row goes on as the tanh, with the cap for a scale
+#pragma unroll
+                for (int i = 0; i < TK; ++i) raw[i] = __float_as_uint(cap_tanh(__uint_as_float(raw[i]) * p.over_cap));
+            }
             // keys [lo, hi) of the block are seen by this row
             const int hi = valid ? pos - kb + 1 : 0;
             const int lo = first_visible_key(pos, p.window, p.chunk) - kb;
@@ -464,7 +470,7 @@ cudaError_t launch_attention_tc(const void* qkv, int qkv_stride, void* out, cons
                                 const int* cu_q, const int* q_start, const int* block_table, int table_stride,
                                 const int* tiles, int n_tiles, int n_pages, int heads, int kv_heads, int head_dim,
                                 int page_size, int window, float scale, int* status, cudaStream_t stream, int chunk,
-                                const float* sinks) {
+                                const float* sinks, float softcap) {
     if (n_tiles == 0) return cudaSuccess;
     if (!attention_tc_supports(head_dim, heads, kv_heads) || page_size % 16 != 0 || tiles == nullptr) return cudaErrorInvalidValue;
     const long long cache_rows = (long long)n_pages * kv_heads * page_size;
@@ -488,7 +494,8 @@ cudaError_t launch_attention_tc(const void* qkv, int qkv_stride, void* out, cons
     p.page_size = page_size;
     p.window = window;
     p.chunk = chunk;
-    p.scale_log2 = scale * 1.4426950408889634f;
+    p.scale_log2 = (softcap > 0.f ? softcap : scale) * 1.4426950408889634f;
+    p.over_cap = softcap > 0.f ? scale / softcap * 2.8853900817779268f : 0.f;
     p.tokens_per_tile = TQ / (heads / kv_heads);
     p.cache_rows = (int)cache_rows;
     p.run_keys = run_keys;
@@ -498,9 +505,11 @@ cudaError_t launch_attention_tc(const void* qkv, int qkv_stride, void* out, cons
     // would fit an SM: each takes all of its tensor memory
     const int halves = head_dim / 64;
     const int smem = max((1 + 2 * 2) * halves * HALF_BYTES + 1024 + 256 + 2 * 128 * 2 * 4, 120 * 1024);
-    auto kernel = head_dim == 128 ? attention_tc_kernel<128> : attention_tc_kernel<64>;
-    static std::atomic<unsigned long long> configured[2] = {{0}, {0}};
-    cudaError_t e = allow_dynamic_smem(kernel, smem, configured[halves - 1]);
+    const bool cap = softcap > 0.f;
+    auto kernel = head_dim == 128 ? (cap ? attention_tc_kernel<128, true> : attention_tc_kernel<128, false>)
+                                  : (cap ? attention_tc_kernel<64, true> : attention_tc_kernel<64, false>);
+    static std::atomic<unsigned long long> configured[4] = {{0}, {0}, {0}, {0}};
+    cudaError_t e = allow_dynamic_smem(kernel, smem, configured[2 * (halves - 1) + (cap ? 1 : 0)]);
     if (e != cudaSuccess) return e;
     return launch(kernel, dim3(n_tiles, kv_heads, 1), dim3(ATC_THREADS, 1, 1), smem, stream, map_k, map_v, p);
 }

@@ -50,6 +50,16 @@ __device__ __forceinline__ int first_visible_key(int pos, int window, int chunk)
     return lo;
 }
 
+// tanh(x) for a score that is capped, given x2 = 2 x log2(e): 1 - 2 / (1 + e^(2x)), the power of two and the reciprocal by the hardware's
+// approximations.  The absolute error stays within a few 2^-22 (near zero the difference cancels, which a cap's absolute scale
+// allows); both ends come out as -1 and 1.
+__device__ __forceinline__ float cap_tanh(float x2) {
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(e) : "f"(x2));
+    asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(r) : "f"(1.f + e));
+    return fmaf(-2.f, r, 1.f);
+}
+
 // The clamped gate of a feed-forward: g = min(gate, limit), u = clamp(up, -limit, limit), g * sigmoid(alpha g) * (u + 1).
 __device__ __forceinline__ float gate_clamp(float g, float u, float alpha, float limit) {
     g = fminf(g, limit);

@@ -303,89 +303,85 @@ cudaError_t launch_layernorm(int out_dtype, float* x, const void* delta, const f
 
 // ------------------------------------------------------------------------- a normed result joins the stream
 
-// One block a row: x += mult * weight * d * rsqrt(mean(d^2) + eps) for the row d of a sublayer's result (a tensor, or the unadded
-// shares of a product, added in the order of their index), all in 32-bit; `out` (or null) takes the new row in the compute dtype,
-// for a sublayer that reads the stream as it is.  Without a delta the row is copied alone.  A thread keeps its first eight
-// values of d in registers; wider rows read the others again.
-template <typename T>
+// One block a row: x += mult * weight * d * rsqrt(mean(d^2) + eps) for the row d of a sublayer's result, all in 32-bit; `out` (or
+// null) takes the new row in the compute dtype, for a sublayer that reads the stream as it is.  D: where d comes from: 0 nowhere (the
+// row is copied alone), 1 a tensor, 2 the unadded shares of a product (added in the order of their index).  A thread has ITEMS times
+// eight values of the row, all in registers: d and x are each read once, and all their loads are on their way together.
+template <typename T, int D, int ITEMS>
 __global__ void __launch_bounds__(512)
 add_normed_kernel(float* __restrict__ x, const T* __restrict__ delta, const float* __restrict__ parts, int n_parts, long long part_stride,
                   const float* __restrict__ weight, float eps, float mult, T* __restrict__ out, int hidden) {
     __shared__ float scratch[32];
     pdl_launch();
-    const int first = threadIdx.x * 8;
-    float w_first[8];
-    if (weight != nullptr && first < hidden) Vec8<float>::load(weight + first, w_first);
     pdl_wait();
     const size_t at = (size_t)blockIdx.x * hidden;
-    auto delta_values = [&](int i, float (&d)[8]) {
-        if (delta) {
-            Vec8<T>::load(delta + at + i, d);
-            return;
-        }
+    const int step = blockDim.x * 8;
+    float d[ITEMS][8], v[ITEMS][8];
+    float ss = 0.f;
 #pragma unroll
-        for (int j = 0; j < 8; ++j) d[j] = 0.f;
+    for (int k = 0; k < ITEMS; ++k) {
+        const int i = threadIdx.x * 8 + k * step;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) d[k][j] = 0.f;
+        if (i >= hidden) continue;
+        Vec8<float>::load(x + at + i, v[k]);
+        if (D == 1) Vec8<T>::load(delta + at + i, d[k]);
+        if (D == 2) {
 #pragma unroll 4
-        for (int q = 0; q < n_parts; ++q) {
-            float e[8];
-            Vec8<float>::load(parts + at + i + q * part_stride, e);
+            for (int q = 0; q < n_parts; ++q) {
+                float e[8];
+                Vec8<float>::load(parts + at + i + q * part_stride, e);
 #pragma unroll
-            for (int j = 0; j < 8; ++j) d[j] += e[j];
-        }
-    };
-    const bool any = delta != nullptr || parts != nullptr;
-    float d0[8], x0[8];
-    float rs = 0.f;
-    if (first < hidden) Vec8<float>::load(x + at + first, x0);
-    if (any) {
-        float ss = 0.f;
-        for (int i = first; i < hidden; i += blockDim.x * 8) {
-            float d[8];
-            delta_values(i, d);
-#pragma unroll
-            for (int j = 0; j < 8; ++j) {
-                ss = fmaf(d[j], d[j], ss);
-                if (i == first) d0[j] = d[j];
+                for (int j = 0; j < 8; ++j) d[k][j] += e[j];
             }
         }
+    }
+    float rs = 0.f;
+    if (D != 0) {
+#pragma unroll
+        for (int k = 0; k < ITEMS; ++k)
+#pragma unroll
+            for (int j = 0; j < 8; ++j) ss = fmaf(d[k][j], d[k][j], ss);
         rs = rsqrtf(block_sum(ss, scratch) / (float)hidden + eps) * mult;
     }
-    for (int i = first; i < hidden; i += blockDim.x * 8) {
-        float v[8];
-        if (i == first) {
 #pragma unroll
-            for (int j = 0; j < 8; ++j) v[j] = x0[j];
-        } else {
-            Vec8<float>::load(x + at + i, v);
+    for (int k = 0; k < ITEMS; ++k) {
+        const int i = threadIdx.x * 8 + k * step;
+        if (i >= hidden) continue;
+        if (D != 0) {
+            float w[8];
+            Vec8<float>::load(weight + i, w);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[k][j] += d[k][j] * rs * w[j];
+            Vec8<float>::store(x + at + i, v[k]);
         }
-        if (any) {
-            float d[8], w[8];
-            if (i == first) {
-#pragma unroll
-                for (int j = 0; j < 8; ++j) { d[j] = d0[j]; w[j] = w_first[j]; }
-            } else {
-                delta_values(i, d);
-                Vec8<float>::load(weight + i, w);
-            }
-#pragma unroll
-            for (int j = 0; j < 8; ++j) v[j] += d[j] * rs * w[j];
-            Vec8<float>::store(x + at + i, v);
-        }
-        if (out) Vec8<T>::store(out + at + i, v);
+        if (out) Vec8<T>::store(out + at + i, v[k]);
     }
 }
 
+template <typename T, int D>
+static cudaError_t launch_add_normed_t(float* x, const void* delta, const float* parts, int n_parts, const float* weight, float eps, float mult,
+                                       void* out, int n_tokens, int hidden, cudaStream_t stream) {
+    const long long part_stride = (long long)n_tokens * hidden;
+    const int eights = hidden / 8;
+    // few rows: as many threads a row as it has eights; many rows: fewer threads with two eights each, so that more rows are at work
+    const int items = eights > 2048 ? 8 : (eights > 1024 ? 4 : (eights > 512 || (n_tokens >= 1024 && eights > 128) ? 2 : 1));
+    const int threads = max(32, ((eights + items - 1) / items + 31) / 32 * 32);
+    if (threads > 512) return cudaErrorInvalidValue;
+    auto kernel = items == 1 ? add_normed_kernel<T, D, 1> : (items == 2 ? add_normed_kernel<T, D, 2>
+                                                                        : (items == 4 ? add_normed_kernel<T, D, 4> : add_normed_kernel<T, D, 8>));
+    return launch(kernel, n_tokens, threads, 0, stream, x, (const T*)delta, parts, n_parts, part_stride, weight, eps, mult, (T*)out, hidden);
+}
+
+// hidden up to 32,768
 cudaError_t launch_add_normed(int dtype, float* x, const void* delta, const float* parts, int n_parts, const float* weight, float eps, float mult,
                               void* out, int n_tokens, int hidden, cudaStream_t stream) {
     if (n_tokens == 0) return cudaSuccess;
     if (hidden % 8 || (delta != nullptr && parts != nullptr) || ((delta != nullptr || parts != nullptr) && weight == nullptr)) return cudaErrorInvalidValue;
-    const int threads = min(512, max(32, ((hidden / 8 + 31) / 32) * 32));
-    const long long part_stride = (long long)n_tokens * hidden;
-    if (dtype == kBF16)
-        return launch(add_normed_kernel<__nv_bfloat16>, n_tokens, threads, 0, stream, x, (const __nv_bfloat16*)delta, parts, n_parts, part_stride,
-                      weight, eps, mult, (__nv_bfloat16*)out, hidden);
-    return launch(add_normed_kernel<float>, n_tokens, threads, 0, stream, x, (const float*)delta, parts, n_parts, part_stride, weight, eps, mult,
-                  (float*)out, hidden);
+    const int d = delta != nullptr ? 1 : (parts != nullptr ? 2 : 0);
+    auto run = dtype == kBF16 ? (d == 0 ? launch_add_normed_t<__nv_bfloat16, 0> : (d == 1 ? launch_add_normed_t<__nv_bfloat16, 1> : launch_add_normed_t<__nv_bfloat16, 2>))
+                              : (d == 0 ? launch_add_normed_t<float, 0> : (d == 1 ? launch_add_normed_t<float, 1> : launch_add_normed_t<float, 2>));
+    return run(x, delta, parts, n_parts, weight, eps, mult, out, n_tokens, hidden, stream);
 }
 
 // ------------------------------------------------------------------------- PolyNorm

@@ -353,7 +353,7 @@ cudaError_t launch_attention_tc(const void* qkv, int qkv_stride, void* out, cons
                                 const int* cu_q, const int* q_start, const int* block_table, int table_stride,
                                 const int* tiles, int n_tiles, int n_pages, int heads, int kv_heads, int head_dim,
                                 int page_size, int window, float scale, int* status, cudaStream_t stream, int chunk = 0,
-                                const float* sinks = nullptr);
+                                const float* sinks = nullptr, float softcap = 0.f);
 
 // Attention of single-token steps: every sequence brings tokens_per_tile = 16 / group tokens at most (one in a
 // decode step).  Grid (sequences, kv_heads, n_splits), four warps a CTA.  With n_splits > 1 the runs' results

@@ -638,11 +638,94 @@ head_norm_gate_wide_kernel(const float* __restrict__ o, const T* __restrict__ y,
     }
 }
 
+// The same, eight values a lane at a time and all of them in registers (ITEMS times eight a lane): a warp (WARPS 1, four pairs a CTA)
+// or a CTA of WARPS warps a (token, head); every column, size and stride a multiple of 8.
+template <typename T, bool GATE_FIRST, int ITEMS, int WARPS>
+__global__ void __launch_bounds__(WARPS == 1 ? 128 : WARPS * 32)
+head_norm_gate_vec_kernel(const float* __restrict__ o, const T* __restrict__ y, int y_stride, int gate_col,
+                          const float* __restrict__ weight, int weight_per_channel, float eps, int act, T* __restrict__ out,
+                          int out_stride, int out_col, float out_scale, const int* __restrict__ token_seq, int n_tokens, int heads,
+                          int v_dim) {
+    __shared__ float sums[WARPS];
+    pdl_launch();
+    pdl_wait();
+    const int lane = WARPS == 1 ? threadIdx.x & 31 : threadIdx.x;
+    const long long pair = WARPS == 1 ? (long long)blockIdx.x * 4 + (threadIdx.x >> 5) : (long long)blockIdx.x;
+    if (pair >= (long long)n_tokens * heads) return;
+    const int t = (int)(pair / heads), h = (int)(pair % heads);
+    constexpr int STEP = WARPS * 32 * 8;
+    T* dst = out + (size_t)t * out_stride + out_col + h * v_dim;
+    if (token_seq != nullptr && token_seq[t] < 0) {     // padding: nothing ran for this token
+        const float zero[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+        for (int i = lane * 8; i < v_dim; i += STEP) Vec8<T>::store(dst + i, zero);
+        return;
+    }
+    const float* src = o + ((size_t)t * heads + h) * v_dim;
+    const T* gate = y + (size_t)t * y_stride + gate_col + h * v_dim;
+    const float* w = weight + (weight_per_channel ? h * v_dim : 0);
+    float v[ITEMS][8], z[ITEMS][8];
+#pragma unroll
+    for (int k = 0; k < ITEMS; ++k) {
+        const int i = lane * 8 + k * STEP;
+        if (i < v_dim) {
+            Vec8<float>::load(src + i, v[k]);
+            Vec8<T>::load(gate + i, z[k]);
+        } else {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[k][j] = z[k][j] = 0.f;
+        }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < ITEMS; ++k)
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            if (GATE_FIRST) v[k][j] = gated(v[k][j], z[k][j], act);
+            ss = fmaf(v[k][j], v[k][j], ss);
+        }
+    ss = warp_sum(ss);
+    if (WARPS > 1) {
+        if ((threadIdx.x & 31) == 0) sums[threadIdx.x >> 5] = ss;
+        __syncthreads();
+        ss = 0.f;
+#pragma unroll
+        for (int k = 0; k < WARPS; ++k) ss += sums[k];
+    }
+    const float r = rsqrtf(ss / (float)v_dim + eps) * out_scale;
+#pragma unroll
+    for (int k = 0; k < ITEMS; ++k) {
+        const int i = lane * 8 + k * STEP;
+        if (i >= v_dim) continue;
+        float u[8];
+        Vec8<float>::load(w + i, u);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            const float n = v[k][j] * r * u[j];
+            u[j] = GATE_FIRST ? n : gated(n, z[k][j], act);
+        }
+        Vec8<T>::store(dst + i, u);
+    }
+}
+
 template <typename T, bool GATE_FIRST>
 static cudaError_t launch_head_norm_gate_t(const float* o, const void* y, int y_stride, int gate_col, const float* weight, int weight_per_channel,
                                            float eps, int act, void* out, int out_stride, int out_col, float out_scale, const int* token_seq,
                                            int n_tokens, int heads, int v_dim, cudaStream_t stream) {
     const long long pairs = (long long)n_tokens * heads;
+    const bool vec = v_dim % 8 == 0 && y_stride % 8 == 0 && gate_col % 8 == 0 && out_stride % 8 == 0 && out_col % 8 == 0 && v_dim <= 8192 &&
+                     (((uintptr_t)o | (uintptr_t)y | (uintptr_t)out | (uintptr_t)weight) & 15) == 0;
+    if (vec) {
+        auto run = [&](auto kernel, int grid, int threads) {
+            return launch(kernel, grid, threads, 0, stream, o, (const T*)y, y_stride, gate_col, weight, weight_per_channel, eps, act, (T*)out,
+                          out_stride, out_col, out_scale, token_seq, n_tokens, heads, v_dim);
+        };
+        const int few = (int)((pairs + 3) / 4);
+        if (v_dim <= 256) return run(head_norm_gate_vec_kernel<T, GATE_FIRST, 1, 1>, few, 128);
+        if (v_dim <= 512) return run(head_norm_gate_vec_kernel<T, GATE_FIRST, 2, 1>, few, 128);
+        if (v_dim <= 1024) return run(head_norm_gate_vec_kernel<T, GATE_FIRST, 1, 4>, (int)pairs, 128);
+        if (v_dim <= 2048) return run(head_norm_gate_vec_kernel<T, GATE_FIRST, 2, 4>, (int)pairs, 128);
+        return run(head_norm_gate_vec_kernel<T, GATE_FIRST, 4, 8>, (int)pairs, 256);
+    }
     if (v_dim >= 1024)
         return launch(head_norm_gate_wide_kernel<T, GATE_FIRST>, (int)pairs, 256, 0, stream, o, (const T*)y, y_stride, gate_col, weight,
                       weight_per_channel, eps, act, (T*)out, out_stride, out_col, out_scale, token_seq, heads, v_dim);

@@ -20,16 +20,47 @@ namespace {
 __device__ __forceinline__ float softplus_all(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float silu_of(float z) { return z / (1.f + expf(-z)); }
 
+__device__ __forceinline__ float silu_fast(float z) {
+    // the power of two and the reciprocal by the hardware's approximations, for a result that is rounded to 16 bits
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(e) : "f"(z * -1.4426950408889634f));
+    asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(r) : "f"(1.f + e));
+    return z * r;
+}
+
+// VEC consecutive values as they lie, fetched ahead of their use.
+template <typename T, int VEC> struct Fetched {
+    T v[VEC];
+    __device__ __forceinline__ void load(const T* p) {
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) v[i] = p[i];
+    }
+    __device__ __forceinline__ float get(int i) const { return to_float(v[i]); }
+};
+template <> struct Fetched<__nv_bfloat16, 4> {
+    uint2 q;
+    __device__ __forceinline__ void load(const __nv_bfloat16* p) { q = *reinterpret_cast<const uint2*>(p); }
+    __device__ __forceinline__ float get(int i) const {
+        const uint32_t w = i < 2 ? q.x : q.y;
+        return __uint_as_float((i & 1) ? (w & 0xffff0000u) : (w << 16));
+    }
+};
+template <> struct Fetched<float, 4> {
+    float4 q;
+    __device__ __forceinline__ void load(const float* p) { q = *reinterpret_cast<const float4*>(p); }
+    __device__ __forceinline__ float get(int i) const { return i == 0 ? q.x : (i == 1 ? q.y : (i == 2 ? q.z : q.w)); }
+};
+
 // VEC consecutive values as floats, and back.
 template <typename T, int VEC> __device__ __forceinline__ void load_values(const T* p, float (&f)[VEC]) {
-    if constexpr (VEC == 8) Vec8<T>::load(p, f);
-    else {
+    Fetched<T, VEC> v;
+    v.load(p);
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) f[i] = to_float(p[i]);
-    }
+    for (int i = 0; i < VEC; ++i) f[i] = v.get(i);
 }
 template <typename T, int VEC> __device__ __forceinline__ void store_values(T* p, const float (&f)[VEC]) {
-    if constexpr (VEC == 8) Vec8<T>::store(p, f);
+    if constexpr (VEC == 4 && sizeof(T) == 2) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]));
+    else if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
     else {
 #pragma unroll
         for (int i = 0; i < VEC; ++i) p[i] = from_float<T>(f[i]);
@@ -46,7 +77,7 @@ template <typename T, int VEC> __device__ __forceinline__ void store_values(T* p
 // tail [rows, taps - 1, channels] (oldest first).  A tile has at least taps - 1 tokens unless it is its sequence's last, so
 // only a sequence's first tile reads the tail, and its threads renew it (each its own channels).
 // With fewer than MAXT taps the missing ones (the oldest) have weight zero.
-template <typename T, int VEC, int MAXT>
+template <typename T, int VEC, int MAXT>      // MAXT at least 2
 __global__ void __launch_bounds__(128)
 causal_conv_kernel(const T* __restrict__ y, int stride, int col, int channels, const float* __restrict__ w, int taps,
                    const float* __restrict__ bias, int act, float* __restrict__ tail, int state_rows, const int* __restrict__ cu_q,
@@ -84,17 +115,22 @@ causal_conv_kernel(const T* __restrict__ y, int stride, int col, int channels, c
         return;
     }
     const T* in = y + col + c0;
-    float before[MAXT][VEC];          // before[j]: the input j places in front of the token (j = 1 .. MAXT - 1)
+    constexpr int PAST = MAXT - 1, AHEAD = 4;
+    float win[PAST + AHEAD][VEC];     // the PAST inputs in front of the present four, and these
 #pragma unroll
-    for (int j = 1; j < MAXT; ++j) {
+    for (int j = 0; j < PAST; ++j) {
 #pragma unroll
-        for (int v = 0; v < VEC; ++v) before[j][v] = 0.f;
-        if (j <= kept) {
-            const int s = a - j;
-            if (s >= t0) load_values<T, VEC>(in + (size_t)s * stride, before[j]);
-            else load_values<float, VEC>(tail + ((size_t)row * kept + kept - (t0 - s)) * channels + c0, before[j]);
+        for (int v = 0; v < VEC; ++v) win[j][v] = 0.f;
+        const int back = PAST - j, s = a - back;
+        if (back <= kept) {
+            if (s >= t0) load_values<T, VEC>(in + (size_t)s * stride, win[j]);
+            else load_values<float, VEC>(tail + ((size_t)row * kept + kept - (t0 - s)) * channels + c0, win[j]);
         }
     }
+    // four tokens' inputs are fetched while the four before them are worked on
+    Fetched<T, VEC> next[AHEAD];
+#pragma unroll
+    for (int k = 0; k < AHEAD; ++k) next[k].load(in + (size_t)min(a + k, e - 1) * stride);
     if (first == 0 && kept > 0) {
         // the kept inputs after the step: its last tokens and, where it brings fewer, what was kept before (a thread reads slot
         // i + n after it has written the slots below i only, so the shift is safe in place)
@@ -108,29 +144,32 @@ causal_conv_kernel(const T* __restrict__ y, int stride, int col, int channels, c
             store_values<float, VEC>(tr + (size_t)i * channels, v);
         }
     }
-    float now[VEC];
-    load_values<T, VEC>(in + (size_t)a * stride, now);
-    for (int t = a; t < e; ++t) {
-        float next[VEC], o[VEC];
-        if (t + 1 < e) load_values<T, VEC>(in + (size_t)(t + 1) * stride, next);
+    for (int t = a; t < e; t += AHEAD) {
 #pragma unroll
-        for (int v = 0; v < VEC; ++v) {
-            float s = b[v];
+        for (int k = 0; k < AHEAD; ++k)
 #pragma unroll
-            for (int j = 0; j < MAXT - 1; ++j) s = fmaf(wt[j][v], before[MAXT - 1 - j][v], s);
-            s = fmaf(wt[MAXT - 1][v], now[v], s);
-            o[v] = act ? silu_of(s) : s;
+            for (int v = 0; v < VEC; ++v) win[PAST + k][v] = next[k].get(v);
+        if (t + AHEAD < e) {
+#pragma unroll
+            for (int k = 0; k < AHEAD; ++k) next[k].load(in + (size_t)min(t + AHEAD + k, e - 1) * stride);
         }
-        store_values<T, VEC>(out + (size_t)t * channels + c0, o);
 #pragma unroll
-        for (int j = MAXT - 1; j >= 2; --j)
+        for (int k = 0; k < AHEAD; ++k) {
+            if (t + k >= e) break;
+            float o[VEC];
 #pragma unroll
-            for (int v = 0; v < VEC; ++v) before[j][v] = before[j - 1][v];
+            for (int v = 0; v < VEC; ++v) {
+                float s = b[v];
 #pragma unroll
-        for (int v = 0; v < VEC; ++v) {
-            if (MAXT > 1) before[1 % MAXT][v] = now[v];
-            now[v] = next[v];
+                for (int j = 0; j < MAXT; ++j) s = fmaf(wt[j][v], win[k + j][v], s);
+                o[v] = !act ? s : (sizeof(T) == 2 ? silu_fast(s) : silu_of(s));
+            }
+            store_values<T, VEC>(out + (size_t)(t + k) * channels + c0, o);
         }
+#pragma unroll
+        for (int j = 0; j < PAST; ++j)
+#pragma unroll
+            for (int v = 0; v < VEC; ++v) win[j][v] = win[AHEAD + j][v];
     }
 }
 
@@ -138,11 +177,11 @@ template <typename T>
 static cudaError_t launch_causal_conv_t(const void* y, int stride, int col, int channels, const float* w, int taps, const float* bias, int act,
                                         float* tail, int state_rows, const int* cu_q, const int* seq_rows, int n_seqs, const int* tiles,
                                         int n_tiles, int per_tile, void* out, int* status, cudaStream_t stream) {
-    const bool vec = stride % 8 == 0 && col % 8 == 0 && channels % 8 == 0 && ((uintptr_t)y & 15) == 0 && ((uintptr_t)out & 15) == 0 &&
+    const bool vec = stride % 4 == 0 && col % 4 == 0 && channels % 4 == 0 && ((uintptr_t)y & 15) == 0 && ((uintptr_t)out & 15) == 0 &&
                      ((uintptr_t)w & 15) == 0 && ((uintptr_t)bias & 15) == 0 && ((uintptr_t)tail & 15) == 0 && taps <= 4;
-    const int per_cta = 128 * (vec ? 8 : 1);
+    const int per_cta = 128 * (vec ? 4 : 1);
     const dim3 grid(n_tiles, (channels + per_cta - 1) / per_cta);
-    auto kernel = vec ? causal_conv_kernel<T, 8, 4> : (taps <= 4 ? causal_conv_kernel<T, 1, 4> : causal_conv_kernel<T, 1, 16>);
+    auto kernel = vec ? causal_conv_kernel<T, 4, 4> : (taps <= 4 ? causal_conv_kernel<T, 1, 4> : causal_conv_kernel<T, 1, 16>);
     return launch(kernel, grid, dim3(128), 0, stream, (const T*)y, stride, col, channels, w, taps, bias, act, tail, state_rows, cu_q, seq_rows,
                   n_seqs, reinterpret_cast<const int2*>(tiles), per_tile, (T*)out, status);
 }

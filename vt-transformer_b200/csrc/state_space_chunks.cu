@@ -3,7 +3,7 @@
 // With l_t = -exp(A_log) d_t, L_t the sum of l over a chunk's tokens up to t, and S_0 the state before the chunk:
 //   y_t  = exp(L_t) S_0^T C_t + sum_{s <= t} (C_t . B_s) exp(L_t - L_s) d_s x_s + D x_t
 //   S'   = exp(L_last) S_0 + sum_s exp(L_last - L_s) d_s B_s x_s^T
-// Two kernels.  The walk goes along a sequence's chunks (a CTA a (sequence, head, 64 columns), the state in the accumulators of
+// Two kernels.  The walk goes along a sequence's chunks (a CTA a (sequence, head, 32 columns), the state in the accumulators of
 // its products) and leaves the state before every chunk; the outputs of all chunks are then formed side by side.
 // In 32-bit: step sizes, their logarithms, sums and exponentials, the state, every sum.  B, C and x are the convolution's bfloat16
 // results; what stands beside them in a product and is 32-bit (the weighted x of the state's update, the state itself) goes in as
@@ -22,6 +22,7 @@ constexpr int kChunk = 64;           // tokens of a chunk
 constexpr int kCols = 64;            // columns of the state (values of a head) a CTA owns
 constexpr int kPad = 8;              // 16-bit numbers between rows in shared memory
 constexpr int kLC = kCols + kPad;
+constexpr int kWalkCols = 32;        // ... in the walk, whose time is the length of its chain: more CTAs, each with less to do
 constexpr int kWalkThreads = 256;
 constexpr int kOutThreads = 128;
 
@@ -44,13 +45,8 @@ struct ChunkArgs {
     int* status;
 };
 
-// d and L of the n tokens from t0 on, for threads 0 .. 63 (two warps, all of whose lanes take part): the step size of this
-// thread's token (0 beyond n) and the sum of the logarithms of the decays up to it; `half_sum` is where the first warp leaves its total.
-__device__ __forceinline__ float step_size(const ChunkArgs& a, int t, bool live, int h, float bias) {
-    if (!live) return 0.f;
-    const float z = __bfloat162float(a.y[(size_t)t * a.stride + a.dt_col + h]) + bias;
-    return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
-}
+__device__ __forceinline__ float softplus_of(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+
 __device__ __forceinline__ float warp_running_sum(float v) {
     const int lane = threadIdx.x & 31;
 #pragma unroll
@@ -72,20 +68,22 @@ __device__ __forceinline__ void split_pair(float v0, float v1, uint32_t& hi, uin
 
 // ------------------------------------------------------------------------- the walk along a sequence's chunks
 
-// Warps: 8 / WN along the state's rows (MT tiles of 16 rows each), WN along the columns.
+// Warps: 8 / WN along the state's rows (MT tiles of 16 rows each), WN along the CTA's 32 columns.  A chunk's step sizes and weights
+// are formed by the first warp, two tokens a lane, while the products of the chunk before run.
 template <int MT, int WN>
 __global__ void __launch_bounds__(kWalkThreads)
 state_space_walk_kernel(const ChunkArgs a) {
-    constexpr int WM = 8 / WN, NP = WM * MT * 16, LN = NP + kPad, NT = 8 / WN;
+    constexpr int WM = 8 / WN, NP = WM * MT * 16, LN = NP + kPad, NT = kWalkCols / 8 / WN, LC = kWalkCols + kPad;
     extern __shared__ __align__(16) unsigned char smem_raw[];
     __nv_bfloat16* bs = reinterpret_cast<__nv_bfloat16*>(smem_raw);          // [2][chunk][LN]
-    __nv_bfloat16* xs = bs + 2 * kChunk * LN;                                // [2][chunk][kLC]
-    __nv_bfloat16* hi = xs + 2 * kChunk * kLC;                               // [chunk][kLC]: weighted x
-    __nv_bfloat16* lo = hi + kChunk * kLC;                                   // [chunk][kLC]: what its rounding left
-    float* ws = reinterpret_cast<float*>(lo + kChunk * kLC);                 // [chunk]: weights; [64] the first warp's sum, [65] the chunk's
+    __nv_bfloat16* xs = bs + 2 * kChunk * LN;                                // [2][chunk][LC]
+    __nv_bfloat16* hi = xs + 2 * kChunk * LC;                                // [chunk][LC]: weighted x
+    __nv_bfloat16* lo = hi + kChunk * LC;                                    // [chunk][LC]: what its rounding left
+    float* ws = reinterpret_cast<float*>(lo + kChunk * LC);                  // [2][chunk]: weights
+    float* all = ws + 2 * kChunk;                                            // [2]: the chunk's whole decay
     pdl_launch();
     const int2 walk = a.walks[blockIdx.x];
-    const int seq = walk.x, h = blockIdx.y, col0 = blockIdx.z * kCols;
+    const int seq = walk.x, h = blockIdx.y, col0 = blockIdx.z * kWalkCols;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, tq = lane & 3;
     const int wm = warp / WN, wn = warp % WN;
     const int dim = a.dim, v_dim = a.v_dim;
@@ -103,21 +101,39 @@ state_space_walk_kernel(const ChunkArgs a) {
     auto load = [&](int tb, int stage) {
         const int n = min(kChunk, t1 - tb);
         __nv_bfloat16* b = bs + stage * kChunk * LN;
-        __nv_bfloat16* x = xs + stage * kChunk * kLC;
+        __nv_bfloat16* x = xs + stage * kChunk * LC;
         for (int c = tid; c < kChunk * (NP / 8); c += kWalkThreads) {
             const int r = c / (NP / 8), i = (c % (NP / 8)) * 8;
             const bool ok = r < n && i < dim;
             cp_async16(b + r * LN + i, a.u + (ok ? (size_t)(tb + r) * a.u_stride + b_col + i : 0), ok);
         }
-        for (int c = tid; c < kChunk * (kCols / 8); c += kWalkThreads) {
-            const int r = c / (kCols / 8), i = (c % (kCols / 8)) * 8;
+        for (int c = tid; c < kChunk * (kWalkCols / 8); c += kWalkThreads) {
+            const int r = c / (kWalkCols / 8), i = (c % (kWalkCols / 8)) * 8;
             const bool ok = r < n && col0 + i < v_dim;
-            cp_async16(x + r * kLC + i, a.u + (ok ? (size_t)(tb + r) * a.u_stride + (size_t)h * v_dim + col0 + i : 0), ok);
+            cp_async16(x + r * LC + i, a.u + (ok ? (size_t)(tb + r) * a.u_stride + (size_t)h * v_dim + col0 + i : 0), ok);
         }
         cp_async_commit();
     };
+    // raw step sizes of tokens 2 lane and 2 lane + 1 of a chunk, fetched a chunk before they are used
+    float raw[2] = {0.f, 0.f};
+    auto fetch = [&](int tb) {
+#pragma unroll
+        for (int k = 0; k < 2; ++k) raw[k] = __bfloat162float(a.y[(size_t)min(tb + 2 * lane + k, t1 - 1) * a.stride + a.dt_col + h]);
+    };
+    auto weigh = [&](int tb, int buf) {
+        float step[2], L[2];
+#pragma unroll
+        for (int k = 0; k < 2; ++k) step[k] = tb + 2 * lane + k < t1 ? softplus_of(raw[k] + bias) : 0.f;
+        const float mine = -rate * step[0] - rate * step[1], sum = warp_running_sum(mine);
+        L[1] = sum;
+        L[0] = sum + rate * step[1];
+        const float last = __shfl_sync(0xffffffffu, sum, 31);
+#pragma unroll
+        for (int k = 0; k < 2; ++k) ws[buf * kChunk + 2 * lane + k] = expf(last - L[k]) * step[k];
+        if (lane == 0) all[buf] = expf(last);
+    };
     load(t0, 0);
-    float step = step_size(a, t0 + tid, tid < kChunk && t0 + tid < t1, h, bias);
+    if (warp == 0) fetch(t0);
     // the state: row (wm MT + m) 16 + gq + 8 i, columns (wn NT + n) 8 + 2 tq and the one behind it
     float* sp = a.state + ((size_t)row * a.heads + h) * dim * v_dim;
     float acc[MT][NT][4];
@@ -145,49 +161,40 @@ state_space_walk_kernel(const ChunkArgs a) {
                         *reinterpret_cast<float2*>(to + (size_t)r * v_dim + c) = make_float2(acc[m][n][2 * i], acc[m][n][2 * i + 1]);
                 }
     };
+    if (warp == 0) {
+        weigh(t0, 0);
+        fetch(min(t0 + kChunk, t1 - 1));
+    }
     const int mat = lane >> 3, r8 = lane & 7;
     int chunk = walk.y, stage = 0;
     for (int tb = t0; tb < t1; tb += kChunk, ++chunk, stage ^= 1) {
-        const bool more = tb + kChunk < t1;
-        if (more) load(tb + kChunk, stage ^ 1);
-        // weights of the chunk's tokens in the state behind it
-        float L = 0.f;
-        if (tid < kChunk) {
-            L = warp_running_sum(-rate * step);
-            if (tid == 31) ws[kChunk] = L;
-        }
-        __syncthreads();
-        if (tid < kChunk) {
-            if (tid >= 32) L += ws[kChunk];
-            if (tid == kChunk - 1) ws[kChunk + 1] = L;
-        }
+        cp_async_wait<0>();
+        __syncthreads();                 // the chunk's rows and weights are there; the products of the chunk before are done
+        if (tb + kChunk < t1) load(tb + kChunk, stage ^ 1);
         keep(a.starts + ((size_t)chunk * a.heads + h) * dim * v_dim);
-        __syncthreads();
-        const float last = ws[kChunk + 1];
-        if (tid < kChunk) {
-            ws[tid] = expf(last - L) * step;
-            const int t = tb + kChunk + tid;
-            step = step_size(a, t, t < t1, h, bias);
-        }
-        if (more) cp_async_wait<1>(); else cp_async_wait<0>();
-        __syncthreads();
-        const __nv_bfloat16* x = xs + stage * kChunk * kLC;
-        for (int e = tid; e < kChunk * (kCols / 2); e += kWalkThreads) {
-            const int r = e / (kCols / 2), i = (e % (kCols / 2)) * 2;
-            const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(x + r * kLC + i));
+        const __nv_bfloat16* x = xs + stage * kChunk * LC;
+        const float* w = ws + stage * kChunk;
+#pragma unroll
+        for (int e = tid; e < kChunk * (kWalkCols / 2); e += kWalkThreads) {
+            const int r = e / (kWalkCols / 2), i = (e % (kWalkCols / 2)) * 2;
+            const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(x + r * LC + i));
             uint32_t vh, vl;
-            split_pair(v.x * ws[r], v.y * ws[r], vh, vl);
-            *reinterpret_cast<uint32_t*>(hi + r * kLC + i) = vh;
-            *reinterpret_cast<uint32_t*>(lo + r * kLC + i) = vl;
+            split_pair(v.x * w[r], v.y * w[r], vh, vl);
+            *reinterpret_cast<uint32_t*>(hi + r * LC + i) = vh;
+            *reinterpret_cast<uint32_t*>(lo + r * LC + i) = vl;
         }
-        const float all = expf(last);
+        const float decay = all[stage];
 #pragma unroll
         for (int m = 0; m < MT; ++m)
 #pragma unroll
             for (int n = 0; n < NT; ++n)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) acc[m][n][e] *= all;
+                for (int e = 0; e < 4; ++e) acc[m][n][e] *= decay;
         __syncthreads();
+        if (warp == 0 && tb + kChunk < t1) {
+            weigh(tb + kChunk, stage ^ 1);
+            fetch(min(tb + 2 * kChunk, t1 - 1));
+        }
         const __nv_bfloat16* b = bs + stage * kChunk * LN;
 #pragma unroll
         for (int k = 0; k < kChunk / 16; ++k) {
@@ -199,7 +206,7 @@ state_space_walk_kernel(const ChunkArgs a) {
 #pragma unroll
             for (int n = 0; n < NT; n += 2) {
                 uint32_t vh[4], vl[4];
-                const size_t at = (size_t)(k * 16 + (mat & 1) * 8 + r8) * kLC + (wn * NT + n) * 8 + (mat >> 1) * 8;
+                const size_t at = (size_t)(k * 16 + (mat & 1) * 8 + r8) * LC + (wn * NT + n) * 8 + (mat >> 1) * 8;
                 ldmatrix_x4_trans(vh, hi + at);
                 ldmatrix_x4_trans(vl, lo + at);
 #pragma unroll
@@ -211,7 +218,6 @@ state_space_walk_kernel(const ChunkArgs a) {
                 }
             }
         }
-        __syncthreads();                 // the stage and the weighted x are done with
     }
     keep(sp);
 }
@@ -258,26 +264,27 @@ state_space_out_kernel(const ChunkArgs a) {
     cp_async_commit();
     float L = 0.f;
     if (tid < kChunk) {
-        const float step = step_size(a, tb + tid, tid < n, h, bias);
+        const float step = tid < n ? softplus_of(__bfloat162float(a.y[(size_t)(tb + tid) * a.stride + a.dt_col + h]) + bias) : 0.f;
         L = warp_running_sum(-rate * step);
         ds[tid] = step;
         if (tid == 31) ds[kChunk] = L;
     }
-    // the state, eight quads a thread at a time
+    // the state: all of a thread's quads on their way together (the products' registers are free yet)
     const float* S = a.starts + ((size_t)blockIdx.x * a.heads + h) * dim * v_dim;
     constexpr int kQuads = NP * (kCols / 4);
-    static_assert(kQuads % (kOutThreads * 4) == 0, "quads of the state a thread");
+    constexpr int kMine = kQuads / kOutThreads, kAtOnce = kMine < 16 ? kMine : 16;
+    static_assert(kQuads % (kOutThreads * kAtOnce) == 0, "quads of the state a thread");
 #pragma unroll 1
-    for (int c0 = tid; c0 < kQuads; c0 += kOutThreads * 4) {
-        float4 v[4];
+    for (int c0 = tid; c0 < kQuads; c0 += kOutThreads * kAtOnce) {
+        float4 v[kAtOnce];
 #pragma unroll
-        for (int k = 0; k < 4; ++k) {
+        for (int k = 0; k < kAtOnce; ++k) {
             const int c = c0 + k * kOutThreads, r = c / (kCols / 4), i = (c % (kCols / 4)) * 4;
             v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
             if (r < dim && col0 + i < v_dim) v[k] = *reinterpret_cast<const float4*>(S + (size_t)r * v_dim + col0 + i);
         }
 #pragma unroll
-        for (int k = 0; k < 4; ++k) {
+        for (int k = 0; k < kAtOnce; ++k) {
             const int c = c0 + k * kOutThreads, r = c / (kCols / 4), i = (c % (kCols / 4)) * 4;
             uint2 vh, vl;
             split_pair(v[k].x, v[k].y, vh.x, vl.x);
@@ -375,10 +382,10 @@ constexpr int kMostBytes = 200 * 1024;
 template <int MT, int WN>
 cudaError_t launch_walk(const ChunkArgs& a, int n, cudaStream_t stream) {
     constexpr int NP = 8 / WN * MT * 16;
-    constexpr int bytes = (2 * kChunk * (NP + kPad) + 4 * kChunk * kLC) * 2 + (kChunk + 4) * 4;
+    constexpr int bytes = (2 * kChunk * (NP + kPad) + 4 * kChunk * (kWalkCols + kPad)) * 2 + (2 * kChunk + 4) * 4;
     static std::atomic<unsigned long long> done{0};
     if (cudaError_t e = allow_dynamic_smem(state_space_walk_kernel<MT, WN>, bytes, done); e != cudaSuccess) return e;
-    return launch(state_space_walk_kernel<MT, WN>, dim3(n, a.heads, (a.v_dim + kCols - 1) / kCols), dim3(kWalkThreads), bytes, stream, a);
+    return launch(state_space_walk_kernel<MT, WN>, dim3(n, a.heads, (a.v_dim + kWalkCols - 1) / kWalkCols), dim3(kWalkThreads), bytes, stream, a);
 }
 
 template <int NP>
@@ -406,8 +413,7 @@ cudaError_t launch_state_space_chunks(const void* u, int u_stride, const void* y
     ChunkArgs a = {(const __nv_bfloat16*)u, u_stride, (const __nv_bfloat16*)y, stride, dt_col, a_log, dt_bias, d, state, state_rows, cu_q, rows,
                    n_seqs, reinterpret_cast<const int2*>(walks), reinterpret_cast<const int2*>(chunks), starts, out, heads, groups, dim, v_dim,
                    status};
-    cudaError_t e = dim <= 32 ? launch_walk<1, 4>(a, n_walks, stream)
-                    : dim <= 64 ? launch_walk<1, 2>(a, n_walks, stream)
+    cudaError_t e = dim <= 64 ? launch_walk<1, 2>(a, n_walks, stream)
                     : dim <= 128 ? launch_walk<1, 1>(a, n_walks, stream)
                                  : launch_walk<2, 1>(a, n_walks, stream);
     if (e != cudaSuccess) return e;

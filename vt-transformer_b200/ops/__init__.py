@@ -289,7 +289,7 @@ def add_normed(x: torch.Tensor, delta, post, out: Optional[torch.Tensor], dtype)
     return x
 
 
-CAUSAL_CONV_TILE = 16            # tokens that a CTA of the convolution over a step's tokens walks (the most taps have 15 before them)
+CAUSAL_CONV_TILE = 32            # tokens that a CTA of the convolution over a step's tokens walks (the most taps have 15 before them)
 
 
 def causal_conv(y, col: int, w: torch.Tensor, bias, tail, ctx, out: torch.Tensor, silu: bool = True, status=None) -> torch.Tensor:
@@ -1014,18 +1014,18 @@ def paged_attention(qkv, out, k_cache, v_cache, ctx, block_table, heads: int, kv
     group = heads // kv_heads
     if sinks is not None or softcap:
         # ``sinks`` [heads] float32: one more term exp(sinks[h]) in the denominator; ``softcap`` c: a score becomes
-        # c tanh(score / c).  The mma.sync kernel takes both: tiles of (token, head of the group) rows for portions, a tile a
-        # sequence in steps of single tokens.
+        # c tanh(score / c).  The mma.sync kernel takes both (tiles of (token, head of the group) rows for portions, a tile a
+        # sequence in steps of single tokens), and so does the tcgen05 kernel for long portions.
         if not tensor_core_attention_takes_extras(qkv.dtype, heads, kv_heads, head_dim, head_dim, k_cache.shape[2]):
             raise ValueError("paged_attention: sinks and capped scores run on the tensor cores in bfloat16 at head sizes that are "
                              "multiples of 16 up to 128; ops.attention_general takes the others")
-        if (not softcap and ATTENTION_KERNEL == "auto" and ctx.max_q_len * group >= 128 and k_cache.shape[2] % 16 == 0
+        if (ATTENTION_KERNEL == "auto" and ctx.max_q_len * group >= 128 and k_cache.shape[2] % 16 == 0
                 and be.attention_tc_supports(head_dim, heads, kv_heads)):
-            # portions long enough to fill tiles of 128 rows, a sink and no cap: the tcgen05 kernel (the sink is the start
-            # of a row's scale and sum there too)
+            # portions long enough to fill tiles of 128 rows: the tcgen05 kernel (the sink is the start of a row's scale and
+            # sum there too; a cap bends a row's scores where they arrive from tensor memory)
             tiles = _attention_tiles(ctx, 128 // group, qkv.device)
             be.attention_tc(qkv, out, k_cache, v_cache, ctx.cu_q, ctx.q_start, block_table, tiles, heads, kv_heads, head_dim, w,
-                            float(scale), status, chunk=c, sinks=sinks)
+                            float(scale), status, chunk=c, sinks=sinks, softcap=float(softcap) if softcap else 0.0)
             return out
         splits, part_o, part_ml = 1, None, None
         if ctx.max_q_len == 1:
