@@ -24,7 +24,7 @@ constexpr int kPad = 8;              // 16-bit numbers between rows in shared me
 constexpr int kLC = kCols + kPad;
 constexpr int kWalkCols = 32;        // ... in the walk, whose time is the length of its chain: more CTAs, each with less to do
 constexpr int kWalkThreads = 256;
-constexpr int kOutThreads = 128;
+constexpr int kOutThreads = 256;
 
 struct ChunkArgs {
     const __nv_bfloat16* u;          // [tokens, u_stride]: x at 0, B at heads * v_dim, C behind it
@@ -224,7 +224,8 @@ state_space_walk_kernel(const ChunkArgs a) {
 
 // ------------------------------------------------------------------------- the outputs of every chunk
 
-// A CTA: a chunk, a head, 64 columns; its four warps 16 tokens each.  NP: the state's rows, padded.
+// A CTA: a chunk, a head, 64 columns; its eight warps 16 tokens and one half of the columns each (the two warps of the same tokens
+// both form their weights).  NP: the state's rows, padded.
 template <int NP>
 __global__ void __launch_bounds__(kOutThreads)
 state_space_out_kernel(const ChunkArgs a) {
@@ -298,12 +299,13 @@ state_space_out_kernel(const ChunkArgs a) {
     cp_async_wait<0>();
     __syncthreads();
 
-    const int mat = lane >> 3, r8 = lane & 7, row0 = warp * 16;
+    const int mat = lane >> 3, r8 = lane & 7, row0 = (warp & 3) * 16, half0 = (warp >> 2) * (kCols / 2);
     if (row0 >= n) return;
     // C's fragments serve both products: with the state and with B
-    float o[kCols / 8][4], s[kChunk / 8][4];
+    constexpr int kTiles = kCols / 16;                  // of eight columns
+    float o[kTiles][4], s[kChunk / 8][4];
 #pragma unroll
-    for (int j = 0; j < kCols / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+    for (int j = 0; j < kTiles; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
 #pragma unroll
     for (int j = 0; j < kChunk / 8; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
 #pragma unroll 2
@@ -311,9 +313,9 @@ state_space_out_kernel(const ChunkArgs a) {
         uint32_t cf[4];
         ldmatrix_x4(cf, cs + (size_t)(row0 + (lane & 7) + ((lane >> 3) & 1) * 8) * LN + k * 16 + (lane >> 4) * 8);
 #pragma unroll
-        for (int j = 0; j < kCols / 8; j += 2) {
+        for (int j = 0; j < kTiles; j += 2) {
             uint32_t vh[4], vl[4];
-            const size_t at = (size_t)(k * 16 + (mat & 1) * 8 + r8) * kLC + j * 8 + (mat >> 1) * 8;
+            const size_t at = (size_t)(k * 16 + (mat & 1) * 8 + r8) * kLC + half0 + j * 8 + (mat >> 1) * 8;
             ldmatrix_x4_trans(vh, sh + at);
             ldmatrix_x4_trans(vl, sl + at);
             mma_bf16(o[j], cf, vl[0], vl[1]);
@@ -334,7 +336,7 @@ state_space_out_kernel(const ChunkArgs a) {
     const float Lr[2] = {Ls[row[0]], Ls[row[1]]};
     const float from[2] = {expf(Lr[0]), expf(Lr[1])};
 #pragma unroll
-    for (int j = 0; j < kCols / 8; ++j)
+    for (int j = 0; j < kTiles; ++j)
 #pragma unroll
         for (int e = 0; e < 4; ++e) o[j][e] *= from[e >> 1];
 #pragma unroll
@@ -353,9 +355,9 @@ state_space_out_kernel(const ChunkArgs a) {
         pf[2] = pack_bf16(s[2 * k + 1][0], s[2 * k + 1][1]);
         pf[3] = pack_bf16(s[2 * k + 1][2], s[2 * k + 1][3]);
 #pragma unroll
-        for (int j = 0; j < kCols / 8; j += 2) {
+        for (int j = 0; j < kTiles; j += 2) {
             uint32_t vf[4];
-            ldmatrix_x4_trans(vf, xs + (size_t)(k * 16 + (mat & 1) * 8 + r8) * kLC + j * 8 + (mat >> 1) * 8);
+            ldmatrix_x4_trans(vf, xs + (size_t)(k * 16 + (mat & 1) * 8 + r8) * kLC + half0 + j * 8 + (mat >> 1) * 8);
             mma_bf16(o[j], pf, vf[0], vf[1]);
             mma_bf16(o[j + 1], pf, vf[2], vf[3]);
         }
@@ -365,8 +367,8 @@ state_space_out_kernel(const ChunkArgs a) {
         if (row[i] >= n) continue;
         float* op = a.out + (size_t)(tb + row[i]) * inner + (size_t)h * v_dim + col0;
 #pragma unroll
-        for (int j = 0; j < kCols / 8; ++j) {
-            const int c = j * 8 + 2 * tq;
+        for (int j = 0; j < kTiles; ++j) {
+            const int c = half0 + j * 8 + 2 * tq;
             if (col0 + c >= v_dim) continue;
             const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(xs + row[i] * kLC + c));
             *reinterpret_cast<float2*>(op + c) = make_float2(fmaf(skip, x.x, o[j][2 * i]), fmaf(skip, x.y, o[j][2 * i + 1]));
