@@ -129,6 +129,123 @@ attention_prepare_kernel(T* __restrict__ y, int stride, int q_col, int k_col, in
     }
 }
 
+// The same without the norm over the whole projection, eight values of a head a lane (dim, half and every column and stride
+// multiples of 8): L lanes a head, the angles' cos and sin once a token in shared memory, the other member of a pair from the lane
+// half / 8 away.
+template <typename T, int L>
+__global__ void __launch_bounds__(256)
+attention_prepare_vec_kernel(T* __restrict__ y, int stride, int q_col, int k_col, int v_col, const int* __restrict__ positions,
+                             const int* __restrict__ token_seq, const float* __restrict__ freq, int half, float norm_eps,
+                             T* __restrict__ k_cache, T* __restrict__ v_cache, const int* __restrict__ block_table,
+                             int table_stride, int n_seqs, int n_pages, int heads, int kv_heads, int dim, int v_dim,
+                             int page_size, int store, int* status, int v_heads, const float* __restrict__ q_weight,
+                             const float* __restrict__ k_weight, int norm_first, float rot_mult, float qt_coef, int qt_every) {
+    __shared__ float2 turn[16 * kMaxPerLane];
+    pdl_launch();
+    const int t = blockIdx.x;
+    const int seq = token_seq[t];
+    const bool seq_ok = seq >= 0 && seq < n_seqs;
+    const int pos = seq_ok ? positions[t] : 0;
+    const int page = (store && seq_ok && pos >= 0) ? block_table[(size_t)seq * table_stride + pos / page_size] : 0;
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        float sn, cs;
+        sincosf((float)pos * freq[i], &sn, &cs);
+        turn[i] = make_float2(cs * rot_mult, sn * rot_mult);
+    }
+    __syncthreads();
+    pdl_wait();
+    if (seq < 0) return;   // padding
+    if (!seq_ok) {
+        if (threadIdx.x == 0) set_status(status, kStatusBadSequence, seq);
+        return;
+    }
+    if (pos < 0) {
+        if (threadIdx.x == 0) set_status(status, kStatusBadPosition, pos);
+        return;
+    }
+    if (store && (page < 0 || page >= n_pages)) {
+        if (threadIdx.x == 0) set_status(status, kStatusBadPage, page);
+        store = 0;
+    }
+    T* row = y + (size_t)t * stride;
+    const int slot = pos % page_size;
+    const int units = heads + (store ? kv_heads : 0);
+    const int lane = threadIdx.x & (L - 1), i0 = lane * 8;
+    const bool live = i0 < dim;
+    const float q_times = qt_coef != 0.f ? 1.f + qt_coef * logf((float)((pos + 1) / qt_every) + 1.f) : 1.f;
+    const int per = 256 / L;
+    // (all lanes of a warp go round equally often: the sums and exchanges below take whole warps)
+    for (int u0 = per * blockIdx.y; u0 < units; u0 += per * gridDim.y) {
+        const int u = u0 + threadIdx.x / L;
+        const bool mine = u < units && live, is_q = u < heads;
+        T* src = row + (is_q ? q_col + u * dim : k_col + (u - heads) * dim);
+        const float* w = is_q ? q_weight : k_weight;
+        float v[8], wv[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) { v[j] = 0.f; wv[j] = 1.f; }
+        if (mine) {
+            Vec8<T>::load(src + i0, v);
+            if (w != nullptr && norm_eps >= 0.f) Vec8<float>::load(w + i0, wv);
+        }
+        auto norm_scale = [&]() {
+            float ss = 0.f;
+#pragma unroll
+            for (int j = 0; j < 8; ++j) ss = fmaf(v[j], v[j], ss);
+#pragma unroll
+            for (int o = L / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+            return rsqrtf(ss / (float)dim + norm_eps);
+        };
+        if (norm_first && norm_eps >= 0.f) {
+            const float sc = norm_scale();
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[j] = v[j] * sc * wv[j];
+        }
+        if (half > 0) {
+            const bool low = i0 < half, turned = i0 < 2 * half;
+            const int other = (threadIdx.x & 31) + (turned ? (low ? half / 8 : -half / 8) : 0);
+            const int f = low ? i0 : i0 - half;
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                const float p = __shfl_sync(0xffffffffu, v[j], other);
+                if (turned) {
+                    const float2 cs = turn[f + j];
+                    v[j] = low ? v[j] * cs.x - p * cs.y : v[j] * cs.x + p * cs.y;
+                }
+            }
+        }
+        float sc = 1.f;
+        if (!norm_first && norm_eps >= 0.f) sc = norm_scale();
+        if (is_q) sc *= q_times;
+        if (!mine) continue;
+        const bool after = !norm_first && norm_eps >= 0.f;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[j] *= after ? sc * wv[j] : sc;
+        Vec8<T>::store((is_q ? src : k_cache + (((size_t)page * kv_heads + (u - heads)) * page_size + slot) * dim) + i0, v);
+    }
+    if (!store) return;
+    for (int e = (threadIdx.x + blockIdx.y * blockDim.x) * 8; e < v_heads * v_dim; e += blockDim.x * gridDim.y * 8) {
+        const int h = e / v_dim, i = e % v_dim;
+        float v[8];
+        Vec8<T>::load(row + v_col + e, v);
+        Vec8<T>::store(v_cache + (((size_t)page * v_heads + h) * page_size + slot) * v_dim + i, v);
+    }
+}
+
+template <typename T>
+static cudaError_t launch_prepare_vec(int lanes, dim3 grid, cudaStream_t stream, T* y, int stride, int q_col, int k_col, int v_col,
+                                      const int* positions, const int* token_seq, const float* freq, int half, float norm_eps, T* k_cache,
+                                      T* v_cache, const int* block_table, int table_stride, int n_seqs, int n_pages, int heads, int kv_heads,
+                                      int dim, int v_dim, int page_size, int store, int* status, int v_heads, const float* q_weight,
+                                      const float* k_weight, int norm_first, float rot_mult, float qt_coef, int qt_every) {
+    auto kernel = lanes <= 2 ? attention_prepare_vec_kernel<T, 2>
+                  : lanes <= 4 ? attention_prepare_vec_kernel<T, 4>
+                  : lanes <= 8 ? attention_prepare_vec_kernel<T, 8>
+                  : lanes <= 16 ? attention_prepare_vec_kernel<T, 16> : attention_prepare_vec_kernel<T, 32>;
+    return launch(kernel, grid, dim3(256), 0, stream, y, stride, q_col, k_col, v_col, positions, token_seq, freq, half, norm_eps, k_cache, v_cache,
+                  block_table, table_stride, n_seqs, n_pages, heads, kv_heads, dim, v_dim, page_size, store, status, v_heads, q_weight,
+                  k_weight, norm_first, rot_mult, qt_coef, qt_every);
+}
+
 cudaError_t launch_attention_prepare(int dtype, void* y, int stride, int q_col, int k_col, int v_col, const int* positions,
                                      const int* token_seq, const float* freq, int half, float norm_eps, void* k_cache,
                                      void* v_cache, const int* block_table, int table_stride, int n_seqs, int n_pages,
@@ -142,6 +259,17 @@ cudaError_t launch_attention_prepare(int dtype, void* y, int stride, int q_col, 
     // projection: a block would write a head of q back while another still adds up the squares of all of them)
     const int slices = (n_tokens >= 1024 || whole) ? 1 : max(1, min(8, (heads + kv_heads + 2 * kPrepareWarps - 1) / (2 * kPrepareWarps)));
     const dim3 grid(n_tokens, slices);
+    const bool vec = !whole && dim % 8 == 0 && half % 8 == 0 && v_dim % 8 == 0 && stride % 8 == 0 && q_col % 8 == 0 && k_col % 8 == 0 && v_col % 8 == 0 &&
+                     (((uintptr_t)y | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)q_weight | (uintptr_t)k_weight) & 15) == 0;
+    if (vec && dtype == kBF16)
+        return launch_prepare_vec<__nv_bfloat16>(dim / 8, grid, stream, (__nv_bfloat16*)y, stride, q_col, k_col, v_col, positions, token_seq, freq,
+                                                 half, norm_eps, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, block_table, table_stride, n_seqs,
+                                                 n_pages, heads, kv_heads, dim, v_dim, page_size, store, status, v_heads, q_weight, k_weight,
+                                                 norm_first, rot_mult, qt_coef, qt_every);
+    if (vec)
+        return launch_prepare_vec<float>(dim / 8, grid, stream, (float*)y, stride, q_col, k_col, v_col, positions, token_seq, freq, half, norm_eps,
+                                         (float*)k_cache, (float*)v_cache, block_table, table_stride, n_seqs, n_pages, heads, kv_heads, dim, v_dim,
+                                         page_size, store, status, v_heads, q_weight, k_weight, norm_first, rot_mult, qt_coef, qt_every);
     if (dtype == kBF16)
         return launch(attention_prepare_kernel<__nv_bfloat16>, grid, 32 * kPrepareWarps, 0, stream, (__nv_bfloat16*)y, stride,
                       q_col, k_col, v_col, positions, token_seq, freq, half, norm_eps, (__nv_bfloat16*)k_cache,
